@@ -34,6 +34,11 @@ typedef struct KronosCudaMatrix KronosCudaMatrix;
 #define KRONOS_CUDA_MATRIX_BIPOLAR 0u /* FusedBipolarLutMatrix, src/kernels/simd_lut.rs:1754-1836 */
 #define KRONOS_CUDA_MATRIX_NF      2u /* NfSdotMatrix (bits 5,4,3; 2 = E8Q2), simd_lut.rs:4796-5226 */
 
+/* Unquantized matrix, row-major little-endian in data0: bits = 16 (bf16) or 32 (fp32), any number of columns; data1, codebook
+ * and scale_group_chunks are ignored.  Accepted by matrix_upload / matrix_image, kronos_cuda_linear (plain y = W x: no
+ * rotation, no quantization of x beyond the matrix's own format) and kronos_cuda_engine_create_blocks.  Not a .k2tb tag. */
+#define KRONOS_CUDA_MATRIX_DENSE   16u
+
 /* Upload flag: reorder gate_up rows from [gate; up] into 64-row [gate_64(ic), up_64(ic)] blocks,
  * as Nibble4SdotMatrix::from_bipolar_with_perm (simd_lut.rs:3297-3327) and
  * NfSdotMatrix::to_gate_up_interleaved (5500-5524) do for the CPU path. */
@@ -231,6 +236,49 @@ KronosCudaEngine *kronos_cuda_engine_create(KronosCudaContext *ctx, const Kronos
                                             size_t n_layers, const float *final_norm,
                                             const KronosCudaMatrixDesc *lm_head, const uint16_t *embed_bf16);
 void kronos_cuda_engine_destroy(KronosCudaEngine *engine);
+
+/* ---- models described block by block (no counterpart in the reference) ---------------------------
+ * Unquantized decoder models whose layers differ in kind: every block names its token mixer, its feed-forward (ff = 0: none)
+ * and its sizes.  x += rms(mixer(x)) * norm1; with ff > 0: x += rms(down(act(up(x)))) * norm2; with side_dim > 0 the per-layer
+ * token input x += rms(side_proj (gelu_tanh(side_gate x) * e)) * side_norm, e = the block's side_dim values of the token's row
+ * of the side embedding table.  rms(v) = v / sqrt(mean(v^2) + rms_norm_eps).  All matrices are KRONOS_CUDA_MATRIX_DENSE with
+ * bits = precision: 16 = bf16 products with fp32 accumulation (residual stream, norms, scores, softmax, recurrent state and
+ * everything that enters a recurrence besides the products stay fp32), 32 = everything fp32.  Embedding tables are bf16. */
+#define KRONOS_CUDA_MIXER_WINDOW_ATTENTION 1u
+#define KRONOS_CUDA_MIXER_GENERAL_DELTA    2u
+
+typedef struct KronosCudaBlocksConfig {
+    uint32_t struct_size;              /* sizeof(KronosCudaBlocksConfig), checked at creation */
+    uint32_t hidden_size, num_blocks, vocab_size, max_seq_len, side_dim, precision;
+    float rms_norm_eps;
+} KronosCudaBlocksConfig;
+
+typedef struct KronosCudaBlockDesc {
+    uint32_t mixer, heads, kv_heads, dim, vdim;
+    uint32_t window;                   /* attention: position i sees 0 <= i - j < window; 0 = every earlier position */
+    uint32_t decay_rank, ff;
+    float decay_scale, unit_eps;       /* delta rule: w = exp(-decay_scale * sigmoid(.)), u = k / sqrt(sum k^2 + unit_eps) */
+    const float *norm1, *norm2;        /* [hidden]; norm2 with ff > 0 */
+    /* attention: per-head RMS norm weights [dim]; score = (q . k) * head_scale[h] - head_slope[h] * (i - j), [heads] each */
+    const float *q_norm, *k_norm, *head_scale, *head_slope;
+    /* delta rule, [heads * dim] each: decay = decay_proj tanh(.) + decay_bias, rate = sigmoid(. + rate_bias), norm weight of o */
+    const float *decay_bias, *rate_bias, *out_norm;
+    const float *act_coef;             /* [4]: act = a N(z) + b N(z^2) + c N(z^3) + e, N = division by the rms over the ff values */
+    const float *side_norm;            /* [hidden] */
+    /* attention: rows q (heads x dim), k (kv_heads x dim), v (kv_heads x vdim); o_proj [hidden][heads * vdim].
+     * delta rule: rows r, k, v, g, a (heads x dim each), then the decay_rank rows that feed tanh; decay_proj
+     * [heads * dim][decay_rank]; o_proj [hidden][heads * dim]. */
+    KronosCudaMatrixDesc in_proj, decay_proj, o_proj, up_proj, down_proj, side_gate, side_proj;
+} KronosCudaBlockDesc;
+
+/* The engine behind the handle is the one above: forward_token_ids, decode_greedy, profile_step, read_hidden, weight_bytes and
+ * destroy serve it.  A forward call at position 0 starts a sequence; any other call continues where the sequence stands
+ * (can_truncate_kv_to says whether a position can be continued from).  save_kv_prefix / restore_kv_prefix copy the whole
+ * sequence (rings and recurrent states) at the position where it stands.  Calls that address the quantized cache fail. */
+KronosCudaEngine *kronos_cuda_engine_create_blocks(KronosCudaContext *ctx, const KronosCudaBlocksConfig *cfg,
+                                                   const KronosCudaBlockDesc *blocks, size_t n_blocks, const float *final_norm,
+                                                   const KronosCudaMatrixDesc *head, const uint16_t *embed_bf16,
+                                                   const uint16_t *side_embed_bf16);
 
 /* MetalLlamaEngine::forward_tokens (metal_gpu.rs:1619-1627): runs n_tok tokens whose embeddings the
  * host supplies (embeds[n_tok][hidden]) at positions pos_start.., writes the logits of the last token

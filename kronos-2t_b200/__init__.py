@@ -10,6 +10,7 @@ from .ffi import (  # noqa: F401
     Matrix,
     MatrixDesc,
     bipolar_desc,
+    dense_desc,
     k2tb_load,
     moe_load,
     k2tb_save,
@@ -19,3 +20,4 @@ from .ffi import (  # noqa: F401
     load_library,
 )
 from .build import build  # noqa: F401
+from .models import generate, load_engine, load_spec  # noqa: F401

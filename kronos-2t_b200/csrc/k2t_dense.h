@@ -1,0 +1,54 @@
+// Dense (unquantized) matrices and their activations: the storage and the matrix products of the block engine
+// (k2t_blocks.cu) and of kronos_cuda_linear on KRONOS_CUDA_MATRIX_DENSE matrices.
+//
+// bf16.  A matrix is cut into PANELS of 64 columns; a panel holds all rows (padded to 128), 128 bytes each, the eight 16-byte
+// chunks of row r stored at chunk position c ^ (r % 8) - the 128-byte swizzle of the tensor-core operand layout, so ANY tile of
+// 8n rows x 64 columns is one contiguous run of the image and one bulk copy puts it into shared memory as a K-major operand.
+// Activations use the same form with tokens for rows (`ld` tokens per panel, a multiple of 8), written in place by the kernels
+// that produce them.  Columns beyond the last are zero in the matrix and finite in the activation.
+// fp32.  Row-major, rows padded to four columns (zeros); activations likewise (`ld` floats per token).
+#pragma once
+#include <cstdint>
+#include <cuda_runtime.h>
+
+#include "k2t_kernels.h"
+
+namespace k2t {
+
+constexpr Format FMT_DENSE16 = static_cast<Format>(16), FMT_DENSE32 = static_cast<Format>(17);
+inline bool is_dense(const MatrixGeom &g) { return g.fmt == FMT_DENSE16 || g.fmt == FMT_DENSE32; }
+
+constexpr uint32_t PANEL = 64;              // columns per panel
+constexpr uint32_t DENSE_ROW_TILE = 128;    // rows are padded to the row tile of the tensor-core kernel
+constexpr uint32_t DENSE_TOK_SLACK = 256;   // a token tile may read this many rows beyond the last panel of an activation
+
+struct Act {                                // activation of a dense product (device memory)
+    void *p;
+    uint32_t ld;                            // bf16: tokens per panel; fp32: floats per token
+};
+
+inline uint32_t dense_panels(uint32_t cols) { return (cols + PANEL - 1) / PANEL; }
+inline uint32_t dense_f32_ld(uint32_t cols) { return (cols + 3u) & ~3u; }
+inline uint32_t act_tokens(uint32_t n_tok) { return (n_tok + 7u) & ~7u; }
+inline uint32_t act_ld(bool f32, uint32_t n_tok, uint32_t cols) { return f32 ? dense_f32_ld(cols) : act_tokens(n_tok); }
+inline size_t act_bytes(bool f32, uint32_t n_tok, uint32_t cols) {
+    return f32 ? (size_t)n_tok * dense_f32_ld(cols) * 4 : ((size_t)dense_panels(cols) * act_tokens(n_tok) + DENSE_TOK_SLACK) * PANEL * 2;
+}
+
+struct DenseView {                          // what the kernels need of a dense matrix
+    const void *base;
+    uint32_t rows, cols, rows_pad, panels;  // fp32: rows_pad = floats per row
+};
+inline DenseView dense_view(const DeviceMatrix &m) {
+    return DenseView{m.d_base, m.geom.rows, m.geom.cols, m.geom.fmt == FMT_DENSE32 ? dense_f32_ld(m.geom.cols) : m.geom.rows_pad, m.geom.nc};
+}
+
+// out[t * out_stride + r] = sum over k of W[r][k] x[t][k], fp32 accumulation.  bf16: up to DENSE_TC_MIN - 1 tokens as weight
+// passes of up to eight tokens, more on the tensor cores; fp32: plain fused multiply-adds.
+constexpr uint32_t DENSE_TC_MIN = 17;
+cudaError_t launch_dense(cudaStream_t s, const DeviceMatrix &m, const Act &x, uint32_t n_tok, float *out, size_t out_stride, int sm_count,
+                         uint32_t *err_flag, uint32_t *launches, bool pdl);
+// fp32 rows [n_tok][cols] -> activation
+cudaError_t launch_dense_pack(cudaStream_t s, bool f32, const float *x, uint32_t n_tok, uint32_t cols, const Act &out, bool pdl);
+
+}  // namespace k2t

@@ -13,127 +13,33 @@
 #include <thread>
 #include <vector>
 
-#include "k2t_context.h"
-#include "k2t_decode_mega.h"
+#include "k2t_blocks.h"
+#include "k2t_dense.h"
+#include "k2t_engine.h"
 #include "k2t_gemv_fused.h"
-#include "k2t_model_kernels.h"
 #include "k2t_prologue.cuh"
-#include "k2t_tp.h"
 
 using namespace k2t;
 
-struct EngineLayer {
-    float *input_norm = nullptr, *post_norm = nullptr, *qkv_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr;
-    KronosCudaMatrix *qkv = nullptr, *o = nullptr, *gate_up = nullptr, *down = nullptr;
-    // sparse-MoE FFN (router + expert records) instead of gate_up / down
-    bool moe = false;
-    float *router_w = nullptr, *router_bias = nullptr;
-    k2t::DeviceMatrix gu_dm{}, dn_dm{};                                // geometry (and image base) of the first expert this rank holds: template of the expert launches
-    uint8_t *d_experts = nullptr;                                     // ONE allocation: the device images of all experts of the layer this rank holds
-    const uint8_t **d_gu_bases = nullptr, **d_dn_bases = nullptr;     // device tables: image base of every expert
-    k2t::ExpertCodebook *d_gu_books = nullptr, *d_dn_books = nullptr; // device tables: decode tables of every expert
-    int gu_fmt = -1, dn_fmt = -1;                                     // kernel format of the layer's experts
-    uint32_t expert0 = 0;                                             // first expert held by this rank (expert parallelism)
-    uint32_t *d_route_ids = nullptr;                                  // [max_batch][32] routes of the last batch
-    float *d_route_w = nullptr;
-    // shared expert of a MoE layer (SharedMoeExpert, sparse_moe.rs:223-315): its matrices live in gate_up / down above
-    uint32_t sh_inter = 0;
-    float *sh_gate_w = nullptr;
-};
+namespace k2t {
 
-struct KronosCudaEngine {
-    KronosCudaContext *ctx = nullptr;
-    KronosCudaEngineConfig cfg{};
-    std::vector<EngineLayer> layers;
-    KronosCudaMatrix *lm_head = nullptr;
-    float *final_norm = nullptr, *rope = nullptr;
-    uint16_t *embed_bf16 = nullptr;
-    // workspace
-    float *hidden = nullptr, *proj = nullptr, *qkv = nullptr, *gate_up = nullptr, *logits = nullptr;
-    int8_t *act_q = nullptr, *q_i8 = nullptr;
-    float *attn_tap = nullptr;                // attention output of the last layer (diagnostic)
-    float *act_s = nullptr, *q_scale = nullptr, *part_m = nullptr, *part_l = nullptr, *part_o = nullptr;
-    float *attn_sc = nullptr, *attn_bmax = nullptr;      // long contexts in CPU order: scores [n_q][kv_stride], block maxima [n_q][kv_stride / 128]
-    bool split_kv = false;                    // long contexts by the split-KV kernels instead (config flag, or the cache is too long for the exact path)
-    int32_t *act_m = nullptr;
-    int8_t *k_q8 = nullptr, *v_q8 = nullptr;
-    int8_t *v_t = nullptr;      // int8 cache without a window: the value rows once more, transposed in 16-position blocks for the value chains
-    float *k_scale = nullptr, *v_scale = nullptr;
-    uint32_t *d_token = nullptr, *d_pos = nullptr, *d_step = nullptr, *d_history = nullptr;
-    uint32_t n_split = 32;
-    uint32_t max_batch = 256;                 // tokens per prompt batch: their projections run on the tensor cores in one weight pass (k2t_gemm_tc.cu), their attention side by side; every per-token buffer holds this many rows (KRONOS_CUDA_PROMPT_BATCH, 16..512)
-    uint32_t ctx_bound = 0;                   // prompt batches (launched eagerly, position known on the host): no token of the batch sees more positions; 0 = size launches for the whole cache
-    uint32_t kv_stride = 0;                   // cache rows per (layer, kv head): the rows the geometry needs (max_seq_len, or sinks + ring) rounded up to 32, so every 32-row tile of rows and scales starts on 16 bytes
-    k2t::KvRing ring{};                       // sliding-window + sink ring (all zero: row = position)
-    uint32_t kv_rows = 0;                     // rows in use per (layer, kv head)
-    // sparse-MoE workspace: normalised hidden state, per-route expert buffers
-    float *x_norm = nullptr, *moe_gu = nullptr, *moe_out = nullptr, *router_logits = nullptr;
-    uint32_t *router_done = nullptr;
-    int8_t *moe_q = nullptr; float *moe_s = nullptr; int32_t *moe_m = nullptr;
-    // shared-expert workspace, [max_batch] rows each: gate_up outputs, the down projection's activation, outputs, gate values
-    uint32_t sh_inter_max = 0;
-    float *sh_gu = nullptr, *sh_out = nullptr, *sh_scale = nullptr;
-    int8_t *sh_q = nullptr; float *sh_s = nullptr; int32_t *sh_m = nullptr;
-    bool has_moe = false;
-    // tensor parallel: exchange buffer (data[2][tp][slot] floats + flags[tp]) and the peers' mappings
-    k2t::TpLink tp{};
-    float *tp_buf = nullptr;
-    uint32_t *tp_done = nullptr;              // CTAs of the current fused exchange that have finished (device word)
-    std::vector<void *> tp_peers;            // mappings opened with cudaIpcOpenMemHandle
-    bool tp_ready = false;
-    float *logits_local = nullptr;            // this rank's logits slice [max_batch][vocab_size]
-    KronosCudaMatrix *embed_matrix = nullptr; // whole lm_head for the token lookup (tied embeddings under tp)
-    uint32_t last_row = 0;                    // row of `hidden` that holds the last forwarded token (prompt batches)
-    bool pdl = true;                          // kernels of a step overlap their prologues with the predecessor's tail
-    bool fused = false;                       // single-token steps: norm / SwiGLU / embedding run as prologues of the GEMV that consumes them (KRONOS_CUDA_FUSED=1)
-    const float *final_hidden = nullptr;      // where the last step left the residual stream of its last token
-    size_t weight_bytes = 0;
-    std::vector<void *> allocs;
-    // whole-token decode kernel (contexts up to ATTN_EXACT_CTX positions)
-    bool mega_ok = false;
-    std::string mega_why;                     // why the kernel is not used, when it is not
-    float *hidden2 = nullptr;
-    k2t::MegaLayer *d_mega_layers = nullptr;
-    k2t::MegaMatrix *d_mega_head = nullptr;
-    uint32_t *d_barrier = nullptr;
-    unsigned long long *d_trace = nullptr;    // phase trace of the last step of the last decode-kernel call
-    uint32_t mega_warp_smem = 0, mega_kmax = 0;
-    size_t mega_smem = 0;
-    cudaGraphExec_t graphs[4] = {nullptr, nullptr, nullptr, nullptr};      // [greedy ? 0 : 1][long context ? 1 : 0] -> 2 * ids + long
-    cudaStream_t graph_stream = nullptr;      // the stream the graphs were captured on
-    // per-kernel-class timing of one step (kronos_cuda_engine_profile_step): while prof_on, every launch is followed
-    // by an event record, so a captured step carries one event node per kernel
-    bool prof_on = false;
-    std::vector<std::pair<const char *, cudaEvent_t>> prof_marks;
+bool engine_count(KronosCudaEngine *e, cudaError_t err, const char *what, uint32_t n) {
+    e->ctx->launches += n;
 #ifdef K2T_TIMELINE
-    std::vector<const char *> tl_labels[4];     // launch labels of the four captured step graphs, in launch order
-    std::vector<const char *> *tl_cur = nullptr;
+    if (e->tl_cur) for (uint32_t i = 0; i < n; ++i) e->tl_cur->push_back(what);
 #endif
-    unsigned long long *d_dbg = nullptr;      // 32 diagnostic words (phase clocks of the attention kernel, layer 0)
-    float *argmax_scratch = nullptr;          // candidates and arrival counter of the argmax kernel
-    bool attn_trace = false;
-};
+    if (e->prof_on && err == cudaSuccess) {
+        cudaEvent_t ev = nullptr;
+        if (!cuda_ok(e->ctx, cudaEventCreate(&ev), "profile event") || !cuda_ok(e->ctx, cudaEventRecord(ev, e->ctx->stream), "profile event"))
+            return false;
+        e->prof_marks.emplace_back(what, ev);
+    }
+    return cuda_ok(e->ctx, err, what);
+}
+
+}  // namespace k2t
 
 namespace {
-
-template <typename T>
-bool dev_alloc(KronosCudaEngine *e, T *&p, size_t count, const T *host = nullptr) {
-    void *raw = nullptr;
-    const size_t bytes = std::max<size_t>(count, 1) * sizeof(T);
-    if (!cuda_ok(e->ctx, cudaMalloc(&raw, bytes), "cudaMalloc(engine)")) return false;
-    e->allocs.push_back(raw);
-    p = static_cast<T *>(raw);
-    if (host) return cuda_ok(e->ctx, cudaMemcpyAsync(p, host, count * sizeof(T), cudaMemcpyHostToDevice, e->ctx->stream), "upload");
-    return cuda_ok(e->ctx, cudaMemsetAsync(p, 0, bytes, e->ctx->stream), "clear");
-}
-
-
-void dev_free(KronosCudaEngine *e, void *p) {
-    if (!p) return;
-    for (size_t i = 0; i < e->allocs.size(); ++i)
-        if (e->allocs[i] == p) { e->allocs.erase(e->allocs.begin() + i); break; }
-    cudaFree(p);
-}
 
 // (Re)builds the KV cache: format `bits` (8 / 4) and geometry - the full causal context, or the sliding-window ring of
 // QuantizedKvCache::new_with_opts (real_llm.rs:1235-1257): taken only when 8 <= window and window + 512 < max_seq_len, sinks
@@ -187,7 +93,7 @@ bool sync_vt(KronosCudaEngine *e) {
 }
 
 // y[t] = W x[t] for the n_tok tokens of the batch (activations [n_tok][cols] in act_*; one weight pass for up to 4 tokens)
-bool count(KronosCudaEngine *e, cudaError_t err, const char *what, uint32_t n = 1);
+bool count(KronosCudaEngine *e, cudaError_t err, const char *what, uint32_t n = 1) { return engine_count(e, err, what, n); }
 
 
 bool gemv_from(KronosCudaEngine *e, const KronosCudaMatrix *m, const int8_t *q, const float *sc, const int32_t *sums, float *out, const char *what,
@@ -201,21 +107,12 @@ bool gemv(KronosCudaEngine *e, const KronosCudaMatrix *m, float *out, const char
     return gemv_from(e, m, e->act_q + act_tok0 * cols, e->act_s + act_tok0 * nc, e->act_m + act_tok0 * nc, out, what, n_tok);
 }
 
-bool count(KronosCudaEngine *e, cudaError_t err, const char *what, uint32_t n) {
-    e->ctx->launches += n;
-#ifdef K2T_TIMELINE
-    if (e->tl_cur) for (uint32_t i = 0; i < n; ++i) e->tl_cur->push_back(what);
-#endif
-    if (e->prof_on && err == cudaSuccess) {
-        cudaEvent_t ev = nullptr;
-        if (!cuda_ok(e->ctx, cudaEventCreate(&ev), "profile event") || !cuda_ok(e->ctx, cudaEventRecord(ev, e->ctx->stream), "profile event"))
-            return false;
-        e->prof_marks.emplace_back(what, ev);
-    }
-    return cuda_ok(e->ctx, err, what);
-}
-
 void fill_embed_args(const KronosCudaEngine *e, EmbedArgs &a);
+
+// calls that address the quantized cache or matrices of the Llama/Qwen layers
+bool quantized_only(KronosCudaEngine *e, const char *call) {
+    return e->blocks == nullptr || fail(e->ctx, std::string(call) + ": not available for an engine made by kronos_cuda_engine_create_blocks");
+}
 
 // tensor parallel: x <- sum over ranks of x (rank order), and the concatenation of the ranks' slices; no-ops on one device
 bool tp_gather(KronosCudaEngine *e, const float *slice, float *all, uint32_t n) {
@@ -246,8 +143,6 @@ bool norm_quant(KronosCudaEngine *e, const float *delta, const float *w, float *
     }
     return count(e, launch_rmsnorm_quant_x(e->ctx->stream, e->hidden, delta, w, c.hidden_size, c.rms_norm_eps, e->act_q, e->act_s, e->act_m, x_norm, T, pdl), "rmsnorm");
 }
-
-enum class Tail { Greedy, LastLogits, AllLogits, None };
 
 bool enqueue_attention(KronosCudaEngine *e, uint32_t l, uint32_t t, uint32_t T, bool long_ctx);
 bool enqueue_attention_batch(KronosCudaEngine *e, uint32_t l, uint32_t T);
@@ -424,6 +319,7 @@ bool enqueue_batch(KronosCudaEngine *e, uint32_t T, bool embed, Tail tail, bool 
     const uint32_t h = c.hidden_size, hd = c.head_dim, q_dim = c.num_attention_heads * hd, inter = c.intermediate_size;
     const uint32_t qkv_rows = q_dim + 2 * c.num_key_value_heads * hd;
     (void)qkv_rows; (void)hd;
+    if (e->blocks) return blocks_enqueue(e, T, embed, tail);
     if (T == 1 && e->fused && tail != Tail::None) return enqueue_fused_step(e, embed, tail, long_ctx);
     e->final_hidden = nullptr;
     if (embed) {
@@ -510,14 +406,17 @@ bool ensure_graphs(KronosCudaEngine *e, size_t warm_pos) {
     // they touch is that position's, which the real step rewrites before anything attends to it, so a prompt already
     // in the cache (and, with a sliding window, every live row of the ring) stays as it is.  Callers set position and
     // token before every replay.
-    const int variants = 2;
+    // Recurrent state has no row to rewrite: it is put aside for the warm-up.
+    const int variants = e->blocks ? 1 : 2;
+    if (e->blocks && !blocks_park_state(e, true)) return false;
     const uint32_t wp = (uint32_t)std::min<size_t>(warm_pos, e->cfg.max_seq_len - 1);
     for (int long_ctx = 0; long_ctx < variants; ++long_ctx)
         if (!set_u32(e, e->d_pos, wp) || !set_u32(e, e->d_token, 0) || !enqueue_batch(e, 1, true, Tail::Greedy, long_ctx != 0) ||
             !sync_and_check(ctx, "engine warm-up step"))
             return false;
+    if (e->blocks && !blocks_park_state(e, false)) return false;
     const uint64_t launches_before = ctx->launches;
-    for (int which = 0; which < 4; ++which) {
+    for (int which = 0; which < 4; which += e->blocks ? 2 : 1) {
         cudaGraph_t graph = nullptr;
         if (!cuda_ok(ctx, cudaStreamBeginCapture(ctx->stream, cudaStreamCaptureModeThreadLocal), "begin capture")) return false;
 #ifdef K2T_TIMELINE
@@ -543,9 +442,10 @@ bool ensure_graphs(KronosCudaEngine *e, size_t warm_pos) {
 
 // the graph of one step: greedy (argmax on the device) or logits only, for the context length this position gives
 cudaGraphExec_t step_graph(const KronosCudaEngine *e, bool greedy, size_t pos) {
-    return e->graphs[(greedy ? 0 : 2) + ((pos + 1 > ATTN_EXACT_CTX || e->ring.window) ? 1 : 0)];
+    return e->graphs[(greedy ? 0 : 2) + (!e->blocks && (pos + 1 > ATTN_EXACT_CTX || e->ring.window) ? 1 : 0)];
 }
 uint32_t step_launches(const KronosCudaEngine *e, size_t pos) {
+    if (e->blocks) return blocks_step_launches(e);
     if (e->fused) {      // lm_head + argmax; per layer qkv, attention (1 or 3 kernels), o, and gate_up / down or norm / router / two expert GEMVs
         uint32_t n = 2;
         for (const EngineLayer &L : e->layers) n += ((pos + 1 > ATTN_EXACT_CTX || e->ring.window) ? 3 : 1) + (L.moe ? 6 : 4);
@@ -745,6 +645,7 @@ void kronos_cuda_engine_destroy(KronosCudaEngine *e) {
     cudaSetDevice(e->ctx->device);
     cudaStreamSynchronize(e->ctx->stream);
     for (cudaGraphExec_t g : e->graphs) if (g) cudaGraphExecDestroy(g);
+    blocks_destroy(e);
     for (EngineLayer &L : e->layers)
     {
         for (KronosCudaMatrix *m : {L.qkv, L.o, L.gate_up, L.down})
@@ -805,7 +706,7 @@ KronosCudaEngine *kronos_cuda_engine_create(KronosCudaContext *ctx, const Kronos
     if (c.tp_size > 1 || c.ep_size > 1) e->fused = false;       // the exchanges of the parallel modes live in the norm kernel
     e->layers.resize(c.num_layers);
     auto bad = [&](const std::string &why) { std::string keep = why; kronos_cuda_engine_destroy(e); fail(ctx, keep); return (KronosCudaEngine *)nullptr; };
-    auto shape_ok = [](const KronosCudaMatrixDesc &d, uint32_t rows, uint32_t cols) { return d.rows == rows && d.cols == cols; };
+    auto shape_ok = [](const KronosCudaMatrixDesc &d, uint32_t rows, uint32_t cols) { return d.rows == rows && d.cols == cols && d.kind != KRONOS_CUDA_MATRIX_DENSE; };
     for (uint32_t l = 0; l < c.num_layers; ++l) {
         const KronosCudaLayerDesc &d = layers[l];
         EngineLayer &L = e->layers[l];
@@ -905,6 +806,7 @@ KronosCudaEngine *kronos_cuda_engine_create(KronosCudaContext *ctx, const Kronos
 
 size_t kronos_cuda_engine_kv_bytes(const KronosCudaEngine *e, size_t positions) {
     if (!e) return 0;
+    if (e->blocks) return blocks_kv_bytes(e, positions);
     // int8 keys and values plus one fp32 scale each per (layer, kv head, position): the reference's
     // 2 * layers * n_kv * (head_dim + 4) bytes per position (real_llm.rs:10223)
     const size_t hd = e->cfg.head_dim, per_head = e->cfg.kv_bits == 4 ? hd / 2 + 2 * (hd / 64) : hd + 4;   // NF4: packed + bf16 per 64
@@ -919,7 +821,7 @@ int32_t kronos_cuda_engine_read_hidden(KronosCudaEngine *e, float *hidden) {
     ctx->err.clear();
     if (!make_current(ctx)) return -1;
     // the final norm kernel has already folded the last down_proj into the residual stream
-    const float *src = e->final_hidden ? e->final_hidden : e->hidden + (size_t)e->last_row * e->cfg.hidden_size;
+    const float *src = e->blocks ? blocks_hidden(e) : e->final_hidden ? e->final_hidden : e->hidden + (size_t)e->last_row * e->cfg.hidden_size;
     if (!cuda_ok(ctx, cudaMemcpyAsync(hidden, src, (size_t)e->cfg.hidden_size * 4,
                                       cudaMemcpyDeviceToHost, ctx->stream), "read hidden") ||
         !sync_and_check(ctx, "read hidden"))
@@ -996,7 +898,8 @@ int32_t kronos_cuda_engine_set_embedding_matrix(KronosCudaEngine *e, const Krono
     if (!e) return -1;
     KronosCudaContext *ctx = e->ctx;
     ctx->err.clear();
-    if (!whole || whole->cols != e->cfg.hidden_size) return fail(ctx, "set_embedding_matrix: the matrix must have hidden_size columns"), -1;
+    if (!quantized_only(e, "set_embedding_matrix")) return -1;
+    if (!whole || whole->kind == KRONOS_CUDA_MATRIX_DENSE || whole->cols != e->cfg.hidden_size) return fail(ctx, "set_embedding_matrix: the matrix must have hidden_size columns"), -1;
     if (e->embed_matrix) { kronos_cuda_matrix_free(ctx, e->embed_matrix); e->embed_matrix = nullptr; }
     e->embed_matrix = kronos_cuda_matrix_upload(ctx, whole, 0);
     for (cudaGraphExec_t &g : e->graphs) if (g) { cudaGraphExecDestroy(g); g = nullptr; }      // captured embed arguments are stale
@@ -1021,6 +924,7 @@ int32_t kronos_cuda_engine_read_attention(KronosCudaEngine *e, float *attention)
     if (!e || !attention) return -1;
     KronosCudaContext *ctx = e->ctx;
     ctx->err.clear();
+    if (!quantized_only(e, "read_attention")) return -1;
     if (!make_current(ctx)) return -1;
     const size_t n = (size_t)e->cfg.num_attention_heads * e->cfg.head_dim;
     if (!cuda_ok(ctx, cudaMemcpyAsync(attention, e->attn_tap, n * 4, cudaMemcpyDeviceToHost, ctx->stream), "read attention") ||
@@ -1048,6 +952,7 @@ int32_t kronos_cuda_engine_read_kv(KronosCudaEngine *e, uint32_t layer, uint32_t
     if (!e) return -1;
     KronosCudaContext *ctx = e->ctx;
     ctx->err.clear();
+    if (!quantized_only(e, "read_kv")) return -1;
     if (!k_q8 || !k_scale || !v_q8 || !v_scale) return fail(ctx, "read_kv: NULL buffer"), -1;
     if (layer >= e->cfg.num_layers || kv_head >= e->cfg.num_key_value_heads || position >= e->cfg.max_seq_len)
         return fail(ctx, "read_kv: index out of range"), -1;
@@ -1068,6 +973,7 @@ int32_t kronos_cuda_engine_read_kv_q4(KronosCudaEngine *e, uint32_t layer, uint3
     if (!e) return -1;
     KronosCudaContext *ctx = e->ctx;
     ctx->err.clear();
+    if (!quantized_only(e, "read_kv_q4")) return -1;
     if (!k_q4 || !k_s16 || !v_q4 || !v_s16) return fail(ctx, "read_kv_q4: NULL buffer"), -1;
     if (layer >= e->cfg.num_layers || kv_head >= e->cfg.num_key_value_heads || position >= e->cfg.max_seq_len)
         return fail(ctx, "read_kv_q4: index out of range"), -1;
@@ -1090,6 +996,7 @@ static size_t kv_row_bytes(const KronosCudaEngine *e) { return e->cfg.kv_bits ==
 static size_t kv_scale_bytes(const KronosCudaEngine *e) { return e->cfg.kv_bits == 4 ? 2 * (e->cfg.head_dim / 64) : 4; }
 
 size_t kronos_cuda_engine_kv_bytes_per_pos(const KronosCudaEngine *e) {
+    if (e && e->blocks) return blocks_kv_bytes(e, 1);
     return e ? 2 * (size_t)e->cfg.num_layers * e->cfg.num_key_value_heads * (kv_row_bytes(e) + kv_scale_bytes(e)) : 0;
 }
 
@@ -1097,6 +1004,7 @@ int64_t kronos_cuda_engine_kv_export(KronosCudaEngine *e, size_t lo, size_t hi, 
     if (!e) return -1;
     KronosCudaContext *ctx = e->ctx;
     ctx->err.clear();
+    if (!quantized_only(e, "kv_export")) return -1;
     if (lo > hi || hi > e->cfg.max_seq_len) return fail(ctx, "kv_export: position range out of bounds"), -1;
     const size_t n = hi - lo, heads = (size_t)e->cfg.num_layers * e->cfg.num_key_value_heads, db = kv_row_bytes(e), sb = kv_scale_bytes(e);
     const size_t total = n * kronos_cuda_engine_kv_bytes_per_pos(e);
@@ -1148,6 +1056,7 @@ int32_t kronos_cuda_engine_kv_import(KronosCudaEngine *e, const uint8_t *data, s
     if (!e) return -1;
     KronosCudaContext *ctx = e->ctx;
     ctx->err.clear();
+    if (!quantized_only(e, "kv_import")) return -1;
     if (n > e->cfg.max_seq_len) return fail(ctx, "kv_import: more positions than max_seq_len"), -1;
     if (n == 0) return 0;
     if (!data || len < n * kronos_cuda_engine_kv_bytes_per_pos(e)) return fail(ctx, "kv_import: blob is shorter than n positions"), -1;
@@ -1198,6 +1107,7 @@ int32_t kronos_cuda_engine_reconfigure_kv(KronosCudaEngine *e, uint32_t kv_bits,
     if (!e) return -1;
     KronosCudaContext *ctx = e->ctx;
     ctx->err.clear();
+    if (!quantized_only(e, "reconfigure_kv")) return -1;
     if (!make_current(ctx) || !cuda_ok(ctx, cudaStreamSynchronize(ctx->stream), "reconfigure_kv")) return -1;
     if (e->cfg.tp_size > 1 || e->cfg.ep_size > 1) {
         if (window != 0) return fail(ctx, "reconfigure_kv: a sliding window is not combined with tensor / expert parallelism"), -1;
@@ -1216,10 +1126,11 @@ int32_t kronos_cuda_engine_kv_sliding_window(const KronosCudaEngine *e, size_t *
     return e->ring.window ? 1 : 0;
 }
 
-size_t kronos_cuda_engine_kv_rows(const KronosCudaEngine *e) { return e ? e->kv_rows : 0; }
+size_t kronos_cuda_engine_kv_rows(const KronosCudaEngine *e) { return e ? e->kv_rows : 0; }      // block models: the longest ring of a layer
 
 int32_t kronos_cuda_engine_can_truncate_kv_to(const KronosCudaEngine *e, size_t cur_pos, size_t target_len) {
     if (!e) return 0;
+    if (e->blocks) return blocks_can_continue(e, target_len) ? 1 : 0;
     if (target_len >= cur_pos) return 1;
     if (e->ring.ring_len > 0) {
         const size_t live = e->ring.window - e->ring.sinks, slack = e->ring.ring_len > live ? e->ring.ring_len - live : 0;
@@ -1236,6 +1147,7 @@ static const char KV_PREFIX_MAGIC[8] = {'K', '2', 'T', 'K', 'V', 'P', 'F', 'X'};
 
 size_t kronos_cuda_engine_kv_prefix_bytes(const KronosCudaEngine *e, size_t n, size_t cur_pos) {
     if (!e) return 0;
+    if (e->blocks) return blocks_snapshot_bytes(e);
     const size_t len = std::min(n, cur_pos), slots = e->ring.ring_len > 0 ? e->kv_rows : std::min<size_t>(len, e->kv_rows);
     const size_t heads = (size_t)e->cfg.num_layers * e->cfg.num_key_value_heads;
     return 32 + 2 * heads * slots * (kv_row_bytes(e) + kv_scale_bytes(e));
@@ -1248,6 +1160,7 @@ int64_t kronos_cuda_engine_save_kv_prefix(KronosCudaEngine *e, size_t n, size_t 
     const size_t total = kronos_cuda_engine_kv_prefix_bytes(e, n, cur_pos);
     if (!out || cap < total) return fail(ctx, "save_kv_prefix: output buffer too small"), -1;
     if (!make_current(ctx)) return -1;
+    if (e->blocks) return blocks_save(e, n, cur_pos, out) ? (int64_t)total : -1;
     const size_t len = std::min(n, cur_pos), slots = e->ring.ring_len > 0 ? e->kv_rows : std::min<size_t>(len, e->kv_rows);
     const size_t heads = (size_t)e->cfg.num_layers * e->cfg.num_key_value_heads, db = kv_row_bytes(e), sb = kv_scale_bytes(e), S = e->kv_stride;
     std::memcpy(out, KV_PREFIX_MAGIC, 8);
@@ -1269,6 +1182,7 @@ int32_t kronos_cuda_engine_restore_kv_prefix(KronosCudaEngine *e, const uint8_t 
     if (!e) return -1;
     KronosCudaContext *ctx = e->ctx;
     ctx->err.clear();
+    if (e->blocks) return data && make_current(ctx) && blocks_restore(e, data, len) ? 0 : -1;
     if (!data || len < 32 || std::memcmp(data, KV_PREFIX_MAGIC, 8) != 0) return fail(ctx, "restore_kv_prefix: not a KV prefix snapshot"), -1;
     uint32_t hdr[6];
     std::memcpy(hdr, data + 8, 24);
@@ -1302,6 +1216,7 @@ static int32_t forward_common(KronosCudaEngine *e, const float *embeds, const ui
     if (tokens)
         for (size_t t = 0; t < n_tok; ++t)
             if (tokens[t] >= (e->cfg.tp_size > 1 ? e->cfg.vocab_total : e->cfg.vocab_size)) return fail(ctx, "forward: token id out of range"), -1;
+    if (e->blocks && !blocks_begin(e, tokens != nullptr, pos_start)) return -1;
     const size_t h = e->cfg.hidden_size, v = e->cfg.tp_size > 1 ? e->cfg.vocab_total : e->cfg.vocab_size;
     if (tokens && n_tok == 1) {         // one decode step: the captured graph
         if (!ensure_graphs(e, pos_start) || !set_u32(e, e->d_pos, (uint32_t)pos_start)) return -1;
@@ -1314,6 +1229,7 @@ static int32_t forward_common(KronosCudaEngine *e, const float *embeds, const ui
             !sync_and_check(ctx, "forward"))
             return -1;
         if (all_logits) std::memcpy(all_logits, last_logits, v * 4);
+        if (e->blocks) blocks_end(e, pos_start + 1);
         return 0;
     }
     // prompt: batches of up to max_batch tokens (forward_prompt / forward_batch_sdot_impl, real_llm.rs:7407-7448, 7450-7860):
@@ -1341,6 +1257,7 @@ static int32_t forward_common(KronosCudaEngine *e, const float *embeds, const ui
         // the token / embedding staging buffers are reused by the next batch: the copies above are stream-ordered
     }
     if (!sync_and_check(ctx, "forward")) return -1;
+    if (e->blocks) blocks_end(e, pos_start + n_tok);
     if (all_logits) std::memcpy(last_logits, all_logits + (n_tok - 1) * v, v * 4);
     return 0;
 }
@@ -1366,6 +1283,7 @@ int32_t kronos_cuda_engine_decode_greedy(KronosCudaEngine *e, uint32_t first_tok
     if (pos_start + n_steps > e->cfg.max_seq_len) return fail(ctx, "decode_greedy: sequence would exceed max_seq_len"), -1;
     if (n_steps == 0) return 0;
     if (!make_current(ctx)) return -1;
+    if (e->blocks && !blocks_begin(e, true, pos_start)) return -1;
     e->last_row = 0;
     if (e->mega_ok && pos_start + n_steps <= ATTN_EXACT_CTX) {
         if (!decode_mega(e, first_token, (uint32_t)pos_start, (uint32_t)n_steps)) return -1;
@@ -1400,6 +1318,7 @@ int32_t kronos_cuda_engine_decode_greedy(KronosCudaEngine *e, uint32_t first_tok
     if (!cuda_ok(ctx, cudaMemcpyAsync(out_tokens, e->d_history, n_steps * 4, cudaMemcpyDeviceToHost, ctx->stream), "copy tokens")) return -1;
     if (last_logits && !cuda_ok(ctx, cudaMemcpyAsync(last_logits, e->logits, vocab_all * 4, cudaMemcpyDeviceToHost, ctx->stream), "copy logits")) return -1;
     if (!sync_and_check(ctx, "decode_greedy")) return -1;
+    if (e->blocks) blocks_end(e, pos_start + n_steps);
 #ifdef K2T_TIMELINE
     if (tl_path) {
         for (auto set : timeline_setters()) set(nullptr);
@@ -1442,6 +1361,7 @@ int64_t kronos_cuda_engine_profile_step(KronosCudaEngine *e, uint32_t token, siz
     // The step is launched kernel by kernel with a timing event after each one (and one in front), without programmatic
     // overlap, so the time between two events is the kernel between them, run alone on a warm device.  A bounded delay
     // kernel keeps the stream busy while the host queues the step, so the gaps between events hold no launch latency.
+    if (e->blocks && !blocks_park_state(e, true)) return -1;
     const bool pdl_was = e->pdl;
     const bool long_ctx = pos + reps > ATTN_EXACT_CTX;
     std::map<std::string, std::pair<double, uint32_t>> acc;
@@ -1484,6 +1404,7 @@ int64_t kronos_cuda_engine_profile_step(KronosCudaEngine *e, uint32_t token, siz
     for (auto &mk : e->prof_marks) cudaEventDestroy(mk.second);
     e->prof_marks.clear();
     if (first) cudaEventDestroy(first);
+    if (e->blocks && !blocks_park_state(e, false)) ok = false;
     if (!ok) return -1;
     std::string out = "kernel class | launches per step | us per step | avg us | share\n";
     char line[256];

@@ -8,6 +8,7 @@
 #include <vector>
 
 #include "k2t_context.h"
+#include "k2t_dense.h"
 #include "k2t_model_kernels.h"
 
 using namespace k2t;
@@ -21,6 +22,7 @@ bool check_gemv_args(KronosCudaContext *ctx, const KronosCudaMatrix *m, const vo
                      const void *xsum, size_t n_tok, const void *out, size_t out_stride) {
     if (!m) return fail(ctx, "gemv: matrix is NULL");
     if (m->device != ctx->device) return fail(ctx, "gemv: matrix lives on another device");
+    if (is_dense(m->dm.geom)) return fail(ctx, "gemv: a dense matrix takes fp32 activations (kronos_cuda_linear)");
     if (!xq || !xs || !out) return fail(ctx, "gemv: NULL buffer");
     if (m->dm.geom.max_odd != 0 && !xsum) return fail(ctx, "gemv: bit-plane matrices need xsum");
     if (n_tok == 0) return fail(ctx, "gemv: n_tok is 0");
@@ -125,6 +127,7 @@ KronosCudaMatrix *kronos_cuda_matrix_upload(KronosCudaContext *ctx, const Kronos
     std::string why;
     if (!matrix_geometry(*desc, g, why)) { fail(ctx, why); return nullptr; }
     const bool interleave = (flags & KRONOS_CUDA_UPLOAD_GATE_UP_INTERLEAVE) != 0;
+    if (interleave && is_dense(g)) { fail(ctx, "gate_up interleaving is not available for dense matrices"); return nullptr; }
     if (interleave && (desc->rows % 128 != 0)) { fail(ctx, "gate_up interleaving requires rows divisible by 128"); return nullptr; }
     if (!make_current(ctx)) return nullptr;
     std::vector<uint8_t> image;
@@ -181,7 +184,7 @@ size_t kronos_cuda_matrix_image(const KronosCudaMatrixDesc *desc, uint32_t flags
     std::string why;
     if (!matrix_geometry(*desc, g, why)) return 0;
     const bool interleave = (flags & KRONOS_CUDA_UPLOAD_GATE_UP_INTERLEAVE) != 0;
-    if (interleave && (desc->rows % 128 != 0)) return 0;
+    if (interleave && (is_dense(g) || desc->rows % 128 != 0)) return 0;
     const size_t need = g.image_bytes();
     if (out && cap >= need) repack_matrix(*desc, g, interleave, out, 4);
     return need;
@@ -288,6 +291,22 @@ static int32_t linear_impl(KronosCudaContext *ctx, const KronosCudaMatrix *m, co
     const MatrixGeom &g = m->dm.geom;
     const size_t n = n_tok * g.cols, nch = n_tok * g.nc, n_out = n_tok * (size_t)g.rows;
     cudaStream_t s = ctx->stream;
+    if (is_dense(g)) {
+        const bool f32 = g.fmt == FMT_DENSE32;
+        if (n_tok > (1u << 20)) return fail(ctx, "linear: too many tokens"), -1;
+        if (!reserve(ctx, ctx->x, n * 4) || !reserve(ctx, ctx->q, act_bytes(f32, (uint32_t)n_tok, g.cols)) || !reserve(ctx, ctx->out, n_out * 4)) return -1;
+        const Act act{ctx->q.p, act_ld(f32, (uint32_t)n_tok, g.cols)};
+        uint32_t launched = 0;
+        // rows that pad the last octet / token tile are read by the products (never stored): keep them finite
+        if (!cuda_ok(ctx, cudaMemcpyAsync(ctx->x.p, x, n * 4, cudaMemcpyHostToDevice, s), "copy x") ||
+            !cuda_ok(ctx, cudaMemsetAsync(ctx->q.p, 0, act_bytes(f32, (uint32_t)n_tok, g.cols), s), "clear activation") ||
+            !cuda_ok(ctx, launch_dense_pack(s, f32, (const float *)ctx->x.p, (uint32_t)n_tok, g.cols, act, false), "dense pack launch") ||
+            !cuda_ok(ctx, launch_dense(s, m->dm, act, (uint32_t)n_tok, (float *)ctx->out.p, g.rows, ctx->sm_count, ctx->d_err, &launched, true), "dense launch") ||
+            !cuda_ok(ctx, cudaMemcpyAsync(out, ctx->out.p, n_out * 4, cudaMemcpyDeviceToHost, s), "copy out"))
+            return -1;
+        ctx->launches += 1 + launched;
+        return !wait || sync_and_check(ctx, "linear") ? 0 : -1;
+    }
     if (!reserve(ctx, ctx->x, n * 4) || !reserve(ctx, ctx->q, n) || !reserve(ctx, ctx->xs, nch * 4) ||
         !reserve(ctx, ctx->xsum, nch * 4) || !reserve(ctx, ctx->out, n_out * 4))
         return -1;

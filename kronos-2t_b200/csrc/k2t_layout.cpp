@@ -1,6 +1,7 @@
 // Host-side repack of reference-format matrices into the device cell-plane layout (k2t_layout.h).
 // Input formats: FusedBipolarLutMatrix (src/kernels/simd_lut.rs:1761-1794) and NfSdotMatrix
 // pair_stream / tail_stream (simd_lut.rs:4850-5023, E8Q2 5118-5226) exactly as stored in .k2tb/.k2tm.
+#include "k2t_dense.h"
 #include "k2t_layout.h"
 
 #include <algorithm>
@@ -104,8 +105,40 @@ inline void put_u16(uint8_t *p, uint16_t v) { p[0] = (uint8_t)(v & 0xFF); p[1] =
 
 }  // namespace
 
+namespace {
+
+// Dense matrices (k2t_dense.h): bf16 panels of 64 columns in the operand swizzle, or row-major fp32.
+bool dense_geometry(const KronosCudaMatrixDesc &d, MatrixGeom &g, std::string &err) {
+    if (d.rows == 0 || d.cols == 0) { err = "dense matrix: no rows or columns"; return false; }
+    if (d.bits != 16 && d.bits != 32) { err = "dense matrix: bits must be 16 (bf16) or 32 (fp32)"; return false; }
+    g.file_bytes = (size_t)d.rows * d.cols * (d.bits / 8);
+    if (!d.data0 || d.len0 != g.file_bytes) { err = "dense matrix: byte count does not match rows x cols"; return false; }
+    g.fmt = d.bits == 16 ? FMT_DENSE16 : FMT_DENSE32;
+    g.rows = d.rows; g.cols = d.cols; g.nc = dense_panels(d.cols);
+    g.rows_pad = d.bits == 16 ? (d.rows + DENSE_ROW_TILE - 1) / DENSE_ROW_TILE * DENSE_ROW_TILE : d.rows;
+    g.image_total = d.bits == 16 ? (size_t)g.nc * g.rows_pad * PANEL * 2 : (size_t)d.rows * dense_f32_ld(d.cols) * 4;
+    return true;
+}
+
+void pack_dense(const KronosCudaMatrixDesc &d, const MatrixGeom &g, uint8_t *out, uint32_t r_lo, uint32_t r_hi) {
+    if (g.fmt == FMT_DENSE32) {
+        const size_t ld = dense_f32_ld(d.cols);
+        for (uint32_t r = r_lo; r < r_hi; ++r) std::memcpy(out + (size_t)r * ld * 4, d.data0 + (size_t)r * d.cols * 4, (size_t)d.cols * 4);
+        return;
+    }
+    for (uint32_t r = r_lo; r < r_hi; ++r)
+        for (uint32_t k = 0; k < d.cols; k += 8) {
+            const uint32_t n = std::min(8u, d.cols - k);
+            uint8_t *dst = out + ((size_t)(k / PANEL) * g.rows_pad + r) * (PANEL * 2) + ((((k / 8) & 7u) ^ (r & 7u)) * 16);
+            std::memcpy(dst, d.data0 + ((size_t)r * d.cols + k) * 2, (size_t)n * 2);
+        }
+}
+
+}  // namespace
+
 bool matrix_geometry(const KronosCudaMatrixDesc &d, MatrixGeom &g, std::string &err) {
     std::memset(&g, 0, sizeof g);
+    if (d.kind == KRONOS_CUDA_MATRIX_DENSE) return dense_geometry(d, g, err);
     if (d.rows == 0 || d.cols == 0 || d.cols % 64 != 0) { err = "matrix: cols must be a positive multiple of 64"; return false; }
     g.rows = d.rows; g.cols = d.cols; g.nc = d.cols / 64;
     const size_t ns = (d.rows + STRIPE - 1) / STRIPE;
@@ -155,7 +188,7 @@ bool matrix_geometry(const KronosCudaMatrixDesc &d, MatrixGeom &g, std::string &
         }
         g.file_bytes = want0 + want1 + 16;
     } else {
-        err = "matrix: unsupported kind (only bipolar=0 and NF=2)";
+        err = "matrix: unsupported kind (bipolar = 0, NF = 2, dense = 16)";
         return false;
     }
     g.rows_pad = (g.rows + 3u) & ~3u;
@@ -174,6 +207,14 @@ bool matrix_geometry(const KronosCudaMatrixDesc &d, MatrixGeom &g, std::string &
 void repack_matrix(const KronosCudaMatrixDesc &d, const MatrixGeom &g, bool interleave, uint8_t *out,
                    unsigned threads) {
     std::memset(out, 0, g.image_bytes());
+    if (is_dense(g)) {
+        const unsigned n_thr = (size_t)d.rows * d.cols < (1u << 20) ? 1u : std::max(1u, std::min(threads, d.rows));
+        const uint32_t per = (d.rows + n_thr - 1) / n_thr;
+        std::vector<std::thread> pool;
+        for (unsigned t = 0; t < n_thr; ++t) pool.emplace_back([&, t] { pack_dense(d, g, out, std::min(d.rows, t * per), std::min(d.rows, (t + 1) * per)); });
+        for (auto &th : pool) th.join();
+        return;
+    }
     const FileView fv(d);
     const uint32_t inter = d.rows / 2;
     // destination row -> source row (gate_up interleave puts gate block ic at rows [128ic, +64), up block at [128ic+64, +64))

@@ -20,6 +20,7 @@
 #include <mutex>
 
 #include "k2t_context.h"
+#include "k2t_dense.h"
 
 using namespace k2t;
 
@@ -59,6 +60,7 @@ extern "C" int32_t kronos_cuda_linear_noalloc(KronosCudaContext *ctx, const Kron
     if (m->device != ctx->device) return fail(ctx, "linear_noalloc: matrix lives on another device"), -1;
     if (!d_x || !d_out) return fail(ctx, "linear_noalloc: NULL buffer"), -1;
     const MatrixGeom &g = m->dm.geom;
+    if (is_dense(g)) return fail(ctx, "linear_noalloc: quantized matrices only (use kronos_cuda_linear)"), -1;
     if (g.cols > kMaxCols)
         return fail(ctx, "linear_noalloc: matrix has " + std::to_string(g.cols) + " columns, the static scratch holds at most " +
                              std::to_string(kMaxCols) + " (use kronos_cuda_linear)"), -1;

@@ -13,6 +13,7 @@ _LIB = None
 
 MATRIX_BIPOLAR = 0
 MATRIX_NF = 2
+MATRIX_DENSE = 16
 UPLOAD_GATE_UP_INTERLEAVE = 1
 
 
@@ -52,6 +53,22 @@ class LayerDesc(C.Structure):
                 ("moe_shared_gate_w", C.c_void_p)]
 
 
+MIXER_WINDOW_ATTENTION, MIXER_GENERAL_DELTA = 1, 2
+
+
+class BlocksConfig(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("struct_size", "hidden_size", "num_blocks", "vocab_size", "max_seq_len", "side_dim", "precision")] + \
+               [("rms_norm_eps", C.c_float)]
+
+
+class BlockDesc(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "window", "decay_rank", "ff")] + \
+               [("decay_scale", C.c_float), ("unit_eps", C.c_float)] + \
+               [(n, C.c_void_p) for n in ("norm1", "norm2", "q_norm", "k_norm", "head_scale", "head_slope", "decay_bias", "rate_bias", "out_norm",
+                                          "act_coef", "side_norm")] + \
+               [(n, MatrixDesc) for n in ("in_proj", "decay_proj", "o_proj", "up_proj", "down_proj", "side_gate", "side_proj")]
+
+
 def load_library():
     """Loads libkronos_cuda.so; raises if it has not been built (no fallback exists)."""
     global _LIB
@@ -89,6 +106,7 @@ def load_library():
     sig("kronos_cuda_gemv_dev", i32, vp, vp, vp, vp, vp, sz, vp, sz, vp)
     sig("kronos_cuda_engine_create", vp, vp, C.POINTER(EngineConfig), vp, C.POINTER(LayerDesc), sz, vp,
         C.POINTER(MatrixDesc), vp)
+    sig("kronos_cuda_engine_create_blocks", vp, vp, C.POINTER(BlocksConfig), C.POINTER(BlockDesc), sz, vp, C.POINTER(MatrixDesc), vp, vp)
     sig("kronos_cuda_engine_destroy", None, vp)
     sig("kronos_cuda_engine_forward_tokens", i32, vp, vp, sz, sz, vp, vp)
     sig("kronos_cuda_engine_forward_token_ids", i32, vp, vp, sz, sz, vp, vp)
@@ -149,6 +167,20 @@ def nf_desc(rows, cols, bits, sgc, codebook, pair_stream, tail_stream):
         desc.codebook[i] = int(cb[i])
     desc._keep = (d0, d1)
     return desc
+
+
+def dense_desc(w, bits):
+    """Unquantized matrix [rows][cols]: bits 16 takes bf16 bit patterns (uint16), bits 32 takes fp32."""
+    d0 = _np(w, np.uint16 if bits == 16 else np.float32)
+    desc = MatrixDesc(kind=MATRIX_DENSE, rows=d0.shape[0], cols=d0.shape[1], bits=bits, data0=d0.ctypes.data, len0=d0.nbytes)
+    desc._keep = (d0,)
+    return desc
+
+
+def bf16_bits(x):
+    """fp32 -> bf16 bit patterns (round to nearest even)."""
+    u = _np(x, np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
 
 
 def matrix_image(desc, gate_up_interleave=False):
@@ -233,6 +265,11 @@ class Context:
         return self._upload(nf_desc(rows, cols, bits, sgc, codebook, pair_stream, tail_stream), rows, cols,
                             gate_up_interleave)
 
+    def upload_dense(self, w, bits):
+        """bf16 bit patterns (bits 16) or fp32 (bits 32), row-major."""
+        desc = dense_desc(w, bits)
+        return self._upload(desc, desc.rows, desc.cols, False)
+
     def _upload(self, desc, rows, cols, interleave):
         h = self.L.kronos_cuda_matrix_upload(self.handle, C.byref(desc), UPLOAD_GATE_UP_INTERLEAVE if interleave else 0)
         if not h:
@@ -314,11 +351,18 @@ def desc_of(m):
 class Engine:
     """Whole-token decode engine (KronosCudaEngine).  `spec`: dict with cfg {hidden, layers, n_q, n_kv, head_dim,
     inter, vocab, max_seq, eps[, qk_norm_after_rope]}, layers [{input_norm, post_norm, qkv_bias, q_norm, k_norm,
-    qkv, o, gate_up, down}], final_norm, lm_head, rope [max_seq][head_dim], embed_bf16 (or None = tied)."""
+    qkv, o, gate_up, down}], final_norm, lm_head, rope [max_seq][head_dim], embed_bf16 (or None = tied).
+
+    A spec with `blocks` describes an unquantized model block by block (kronos_cuda_engine_create_blocks): cfg {hidden, vocab,
+    max_seq, eps, side_dim, precision 16 | 32}, blocks [{mixer, heads, dim, .. as the fields of KronosCudaBlockDesc; vectors fp32,
+    matrices bf16 bit patterns (precision 16) or fp32}], final_norm, head, embed and side_embed (bf16 bit patterns)."""
 
     def __init__(self, ctx, spec):
         self.ctx, self.L = ctx, ctx.L
         c = spec["cfg"]
+        if "blocks" in spec:
+            self._create_blocks(spec)
+            return
         self.cfg = EngineConfig(C.sizeof(EngineConfig), c["hidden"], c["layers"], c["n_q"], c["n_kv"], c["head_dim"], c["inter"], c["vocab"],
                                 c["max_seq"], c["eps"], int(c.get("qk_norm_after_rope", 0)), int(c.get("kv_bits", 8)))
         self.cfg.kv_window, self.cfg.kv_sinks = int(c.get("kv_window", 0)), int(c.get("kv_sinks", 0))
@@ -378,6 +422,30 @@ class Engine:
         if spec.get("embed_matrix") is not None:
             md = desc_of(spec["embed_matrix"])
             self.ctx._check(self.L.kronos_cuda_engine_set_embedding_matrix(self.handle, C.byref(md)))
+
+    def _create_blocks(self, spec):
+        c, keep = spec["cfg"], []
+        self.cfg = BlocksConfig(C.sizeof(BlocksConfig), c["hidden"], len(spec["blocks"]), c["vocab"], c["max_seq"], c.get("side_dim", 0), c["precision"], c["eps"])
+        self.vocab = c["vocab"]
+
+        def fill(d, field, value):
+            if isinstance(getattr(d, field), MatrixDesc):
+                value = dense_desc(value, c["precision"])
+                keep.append(value)
+            elif isinstance(value, np.ndarray):
+                keep.append(_np(value, np.float32))
+                value = keep[-1].ctypes.data
+            setattr(d, field, value)
+
+        blocks = (BlockDesc * len(spec["blocks"]))()
+        for d, b in zip(blocks, spec["blocks"]):
+            for field, value in b.items():
+                fill(d, field, value)
+        head, fn, emb = dense_desc(spec["head"], c["precision"]), _np(spec["final_norm"], np.float32), _np(spec["embed"], np.uint16)
+        side = None if spec.get("side_embed") is None else _np(spec["side_embed"], np.uint16)
+        self.handle = self.L.kronos_cuda_engine_create_blocks(self.ctx.handle, C.byref(self.cfg), blocks, len(spec["blocks"]), _p(fn), C.byref(head), _p(emb), _p(side))
+        if not self.handle:
+            raise KronosCudaError(self.L.kronos_cuda_last_error(self.ctx.handle).decode())
 
     def tp_handle(self):
         """This rank's 64-byte inter-process handle of its exchange buffer."""

@@ -1,0 +1,157 @@
+"""Model folders: config.json chooses the architecture, the architecture's reader turns config and weights into an engine spec
+(the dictionary `Engine` takes).
+
+    spec = load_spec(folder, dtype="bfloat16", max_seq=4096)
+    engine = load_engine(ctx, folder)
+
+Registered: `Folizen` (config.json + model.safetensors: blocks of sliding-window attention and generalized delta rule), and the
+compiled Llama / Qwen models (a Hugging Face config.json beside one .k2tb container)."""
+import glob
+import json
+import mmap
+import os
+
+import numpy as np
+
+from . import ffi
+
+READERS = {}
+
+
+def register(*names):
+    def add(fn):
+        for n in names:
+            READERS[n] = fn
+        return fn
+    return add
+
+
+def read_config(folder):
+    with open(os.path.join(folder, "config.json")) as f:
+        return json.load(f)
+
+
+def architecture(config):
+    """The registered name a config.json asks for (`architecture`, or the first known entry of `architectures`)."""
+    names = [config["architecture"]] if "architecture" in config else config.get("architectures", [])
+    for n in names:
+        if n in READERS:
+            return n
+    raise ValueError(f"no reader for the architecture {names or 'of this config.json'}; known: {', '.join(sorted(READERS))}")
+
+
+def load_spec(folder, dtype="bfloat16", max_seq=4096):
+    if dtype not in ("bfloat16", "float32"):
+        raise ValueError("dtype must be bfloat16 or float32")
+    config = read_config(folder)
+    return READERS[architecture(config)](folder, config, dtype, max_seq)
+
+
+def load_engine(ctx, folder, dtype="bfloat16", max_seq=4096):
+    return ffi.Engine(ctx, load_spec(folder, dtype, max_seq))
+
+
+def generate(engine, prompt, n_steps):
+    """Greedy continuation: the prompt in batches, then the device-side decode loop.  Returns the new token ids."""
+    prompt = np.asarray(prompt, np.uint32)
+    if len(prompt) > 1:
+        engine.forward_token_ids(prompt[:-1])
+    return engine.decode_greedy(int(prompt[-1]), len(prompt) - 1, n_steps)
+
+
+# ---- safetensors: 8-byte little-endian header length, JSON {name: {dtype, shape, data_offsets}}, data
+_SAFE_DTYPES = {"BF16": np.uint16, "F32": np.float32, "F16": np.float16, "I32": np.int32, "I64": np.int64, "U8": np.uint8}
+
+
+class Tensors:
+    """Tensors of a safetensors file, mapped; bf16 ones come as bit patterns (`bits`) or widened to fp32 (`f32`)."""
+
+    def __init__(self, path):
+        with open(path, "rb") as f:
+            self._map = mmap.mmap(f.fileno(), 0, access=mmap.ACCESS_READ)
+        n = int.from_bytes(self._map[:8], "little")
+        self._base = 8 + n
+        self._info = {k: v for k, v in json.loads(self._map[8:8 + n]).items() if k != "__metadata__"}
+
+    def __contains__(self, name):
+        return name in self._info
+
+    def shape(self, name):
+        return tuple(self._info[name]["shape"])
+
+    def raw(self, name):
+        t = self._info[name]
+        lo, hi = t["data_offsets"]
+        dt = np.dtype(_SAFE_DTYPES[t["dtype"]]).newbyteorder("<")
+        return np.frombuffer(self._map, dt, (hi - lo) // dt.itemsize, self._base + lo).reshape(t["shape"])
+
+    def f32(self, name):
+        a = self.raw(name)
+        if self._info[name]["dtype"] == "BF16":
+            return (a.astype(np.uint32) << 16).view(np.float32)
+        return a.astype(np.float32)
+
+    def bits(self, name):
+        return self.raw(name) if self._info[name]["dtype"] == "BF16" else ffi.bf16_bits(self.f32(name))
+
+
+# ---- Folizen
+DELTA_DECAY_SCALE = float(np.exp(-0.5))     # log-decay of a key channel = -exp(-1/2) sigmoid(.)
+DELTA_UNIT_EPS = 1e-6
+
+
+def alibi_slopes(heads):
+    return np.array([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], np.float32)
+
+
+@register("Folizen")
+def folizen_spec(folder, config, dtype, max_seq):
+    t = Tensors(os.path.join(folder, "model.safetensors"))
+    mat = t.bits if dtype == "bfloat16" else t.f32
+
+    def rows(*names):
+        return np.concatenate([mat(n) for n in names])
+
+    side = (config.get("token_side") or {}).get("dim", 0)
+    blocks = []
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        x = p + "mix."
+        b = dict(heads=m["heads"], dim=m["dim"], norm1=t.f32(p + "norm1"), o_proj=mat(x + "o"))
+        if layer["type"] == "attention":
+            b.update(mixer=ffi.MIXER_WINDOW_ATTENTION, kv_heads=m["kv_heads"], vdim=m["vdim"], window=(m.get("mask") or {}).get("size", 0),
+                     q_norm=t.f32(x + "q.norm"), k_norm=t.f32(x + "k.norm"), head_scale=np.float32(m["scale"]) * t.f32(x + "temp"),
+                     head_slope=alibi_slopes(m["heads"]), in_proj=rows(x + "q", x + "k", x + "v"))
+        elif layer["type"] == "general_delta":
+            b.update(mixer=ffi.MIXER_GENERAL_DELTA, decay_rank=t.shape(x + "w1")[0], decay_scale=DELTA_DECAY_SCALE, unit_eps=DELTA_UNIT_EPS,
+                     decay_bias=t.f32(x + "w0"), rate_bias=t.f32(x + "a.b"), out_norm=t.f32(x + "norm"), decay_proj=mat(x + "w2"),
+                     in_proj=rows(x + "r", x + "k", x + "v", x + "g", x + "a", x + "w1"))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        if layer.get("mlp") is not None:
+            if layer["mlp"].get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {layer['mlp']['kind']!r}")
+            b.update(ff=t.shape(p + "mlp.up")[0], norm2=t.f32(p + "norm2"), act_coef=t.f32(p + "mlp.act"), up_proj=mat(p + "mlp.up"), down_proj=mat(p + "mlp.down"))
+        if side:
+            b.update(side_norm=t.f32(p + "side.norm"), side_gate=mat(p + "side.gate"), side_proj=mat(p + "side.proj"))
+        blocks.append(b)
+    vocab, width = t.shape("embed")
+    return dict(cfg=dict(hidden=width, vocab=vocab, max_seq=max_seq, eps=config["norm"]["eps"], side_dim=side, precision=16 if dtype == "bfloat16" else 32),
+                blocks=blocks, final_norm=t.f32("final.norm"), head=mat("head"), embed=t.bits("embed"), side_embed=t.bits("side.embed") if side else None)
+
+
+# ---- compiled Llama / Qwen models
+@register("LlamaForCausalLM", "Qwen2ForCausalLM", "Qwen3ForCausalLM")
+def compiled_spec(folder, config, dtype, max_seq):
+    """A .k2tb container with the model's Hugging Face config.json (the container holds no shapes)."""
+    from . import synth
+    if dtype != "bfloat16":
+        raise ValueError("compiled models run in their quantized format")
+    files = sorted(glob.glob(os.path.join(folder, "*.k2tb")))
+    if len(files) != 1:
+        raise ValueError(f"{folder}: one .k2tb container is needed, found {len(files)}")
+    heads = config["num_attention_heads"]
+    hd = config.get("head_dim") or config["hidden_size"] // heads
+    cfg = dict(hidden=config["hidden_size"], n_q=heads, n_kv=config.get("num_key_value_heads", heads), head_dim=hd, inter=config["intermediate_size"],
+               vocab=config["vocab_size"], max_seq=max_seq, eps=config.get("rms_norm_eps", 1e-5))
+    return ffi.k2tb_load(files[0], cfg, synth.rope_table(max_seq, hd, config.get("rope_theta", 10000.0)))[0]

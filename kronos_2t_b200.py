@@ -11,3 +11,8 @@ _spec = importlib.util.spec_from_file_location(
 _mod = importlib.util.module_from_spec(_spec)
 sys.modules["kronos_2t_b200"] = _mod
 _spec.loader.exec_module(_mod)
+
+if __name__ == "__main__":
+    from kronos_2t_b200.cli import main
+
+    main()
