@@ -17,12 +17,14 @@ namespace k2t {
 namespace {
 
 __device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(-x)); }
+// Decays are kept as w - 1: a channel that decays by a hair per token would lose that hair in the rounding of w, the same way
+// at every token, and a state carried over thousands of tokens would show it.
+__device__ __forceinline__ float decay_minus_one(float scale, float logit) { return expm1f(-scale * sigmoidf(logit)); }
 
 // ---- packed fp32 pairs
 __device__ __forceinline__ uint64_t pk(float a, float b) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
 __device__ __forceinline__ void upk(uint64_t v, float &a, float &b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
 __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) { uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
 __device__ __forceinline__ ulonglong2 lds2(uint32_t saddr) {
     ulonglong2 v;
     asm volatile("ld.shared.v2.u64 {%0, %1}, [%2];" : "=l"(v.x), "=l"(v.y) : "r"(saddr));
@@ -72,7 +74,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
         const float z = row_dot8<F32>(a.decay, c, 0, a.decay.panels, s_t, sub) + __ldg(a.decay_bias + c);
         if (i < dim && sub == 0) {
             const float u = s_k[i] * inv_k;
-            s_w[i] = expf(-a.decay_scale * sigmoidf(z));
+            s_w[i] = decay_minus_one(a.decay_scale, z);
             s_u[i] = u;
             s_au[i] = sigmoidf(__ldcg(in + 4 * HD + i) + __ldg(a.rate_bias + c)) * u;
         }
@@ -100,8 +102,8 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
         for (uint32_t i = 0; i < ST_KEYS; ++i) {
             const uint32_t key = sl * ST_KEYS + i;
             const float w = s_w[key], au = -s_au[key], k = s_k[key], r = s_r[key];
-            st[i].x = __fmaf_rn(au, c.x, __fmaf_rn(w, st[i].x, k * v.x)); st[i].y = __fmaf_rn(au, c.y, __fmaf_rn(w, st[i].y, k * v.y));
-            st[i].z = __fmaf_rn(au, c.z, __fmaf_rn(w, st[i].z, k * v.z)); st[i].w = __fmaf_rn(au, c.w, __fmaf_rn(w, st[i].w, k * v.w));
+            st[i].x = __fmaf_rn(au, c.x, __fmaf_rn(w, st[i].x, __fmaf_rn(k, v.x, st[i].x))); st[i].y = __fmaf_rn(au, c.y, __fmaf_rn(w, st[i].y, __fmaf_rn(k, v.y, st[i].y)));
+            st[i].z = __fmaf_rn(au, c.z, __fmaf_rn(w, st[i].z, __fmaf_rn(k, v.z, st[i].z))); st[i].w = __fmaf_rn(au, c.w, __fmaf_rn(w, st[i].w, __fmaf_rn(k, v.w, st[i].w)));
             o.x = __fmaf_rn(r, st[i].x, o.x); o.y = __fmaf_rn(r, st[i].y, o.y); o.z = __fmaf_rn(r, st[i].z, o.z); o.w = __fmaf_rn(r, st[i].w, o.w);
             *reinterpret_cast<float4 *>(state + (size_t)i * D) = st[i];
         }
@@ -132,7 +134,7 @@ __global__ void __launch_bounds__(256) delta_tanh_kernel(const float *__restrict
     act_store<F32>(out, i / rank, i % rank, tanhf(__ldcg(in + (i / rank) * in_stride + i % rank)));
 }
 
-// one warp per (token, head): record [w | a u | u | k | r | v], drow floats each
+// one warp per (token, head): record [w - 1 | a u | u | k | r | v], drow floats each
 __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a, uint32_t n_tok) {
     const uint32_t lane = threadIdx.x & 31, h = blockIdx.y, t = blockIdx.x * 8 + (threadIdx.x >> 5), D = a.drow, dim = a.dim, HD = a.heads * dim;
     pdl_wait();
@@ -148,7 +150,7 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a, uint
         if (i < dim) {
             k = __ldcg(in + HD + i);
             u = k * inv_k;
-            w = expf(-a.decay_scale * sigmoidf(__ldcg(lg + i) + __ldg(a.decay_bias + h * dim + i)));
+            w = decay_minus_one(a.decay_scale, __ldcg(lg + i) + __ldg(a.decay_bias + h * dim + i));
             au = sigmoidf(__ldcg(in + 4 * HD + i) + __ldg(a.rate_bias + h * dim + i)) * u;
             r = __ldcg(in + i);
             v = __ldcg(in + 2 * HD + i);
@@ -219,8 +221,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float *__restrict
 #pragma unroll
             for (int i = 0; i < KI; ++i) {          // w S + k v^T does not need the reduced product
                 const ulonglong2 w = lds2(ak + i * 128), k = lds2(ak + 3 * D * 4 + i * 128);
-                s[i][0] = fma2(w.x, s[i][0], mul2(k.x, v2));
-                s[i][1] = fma2(w.y, s[i][1], mul2(k.y, v2));
+                s[i][0] = fma2(w.x, s[i][0], fma2(k.x, v2, s[i][0]));
+                s[i][1] = fma2(w.y, s[i][1], fma2(k.y, v2, s[i][1]));
             }
             float e0, e1, e2, e3;
             upk(d0, e0, e1);

@@ -86,7 +86,7 @@ def same(a, b):
 
 
 @pytest.mark.parametrize("name,cls_name", [("KronosCudaMatrixDesc", "MatrixDesc"), ("KronosCudaEngineConfig", "EngineConfig"),
-                                           ("KronosCudaLayerDesc", "LayerDesc")])
+                                           ("KronosCudaLayerDesc", "LayerDesc"), ("KronosCudaBlocksConfig", "BlocksConfig"), ("KronosCudaBlockDesc", "BlockDesc")])
 def test_struct_layouts_agree(name, cls_name):
     from kronos_2t_b200 import ffi
     h, r, c = header_struct(name), rust_struct(name), ctypes_struct(getattr(ffi, cls_name))
