@@ -921,6 +921,110 @@ def run_decode_only(args, local_rank):
     ctx.close()
 
 
+def _folizen_bytes(c, n_layers, ctx_len):
+    """(weight bytes, cache + state bytes) one decoded token of a block model streams."""
+    h, hd, kv = c["hidden"], c["heads"] * c["dim"], c["kv_heads"] * c["dim"]
+    side = 2 * c["side_dim"] * h
+    attn, delta = (hd + 2 * kv) * h + h * hd + 2 * c["ff"] * h + side, (5 * hd + c["rank"]) * h + hd * c["rank"] + h * hd + side
+    na, nd = (n_layers + 1) // 2, n_layers // 2
+    return 2 * (na * attn + nd * delta + c["vocab"] * h), na * 2 * min(ctx_len, c["window"]) * kv * 2 + nd * 2 * c["heads"] * c["dim"] ** 2 * 4
+
+
+def _folizen_flops(c, n_layers):
+    """2 x multiply-adds of one prompt token's projections (head left out)."""
+    h, hd, kv = c["hidden"], c["heads"] * c["dim"], c["kv_heads"] * c["dim"]
+    side = 2 * c["side_dim"] * h
+    attn, delta = (hd + 2 * kv) * h + h * hd + 2 * c["ff"] * h + side, (5 * hd + c["rank"]) * h + hd * c["rank"] + h * hd + side
+    return 2 * ((n_layers + 1) // 2 * attn + n_layers // 2 * delta)
+
+
+def run_folizen(args, local_rank):
+    """Block models (random bf16 weights): prompt and decode throughput at real layer sizes, beside a Llama shape of the same
+    width, depth, heads and MLP on the quantized engine (nf4g128 weights, int8 cache)."""
+    import numpy as np
+    import torch
+    import kronos_2t_b200 as k2
+    from kronos_2t_b200 import synth
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device (there is no CPU fallback)")
+    ctx = k2.Context(local_rank)
+    stream = torch.cuda.Stream(device=local_rank)
+    torch.cuda.set_stream(stream)
+    ctx.set_stream(stream.cuda_stream)
+    peak, peak_kind = peaks()
+    with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+        tf_peak = float(json.load(f)["bf16_tflops_sustained"])
+    rng = np.random.Generator(np.random.PCG64(31))
+
+    def timed(fn, reps=3):
+        best = None
+        for _ in range(reps):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            e0.record(stream)
+            fn()
+            e1.record(stream)
+            torch.cuda.synchronize()
+            best = e0.elapsed_time(e1) if best is None else min(best, e0.elapsed_time(e1))
+        return best
+
+    out = {"mode": "folizen", "peak_kind": peak_kind, "data": "synthetic (random weights)", "models": []}
+    steps = args.folizen_steps
+    sampler = ClockSampler(local_rank)
+    sampler.start()
+    for name in (args.folizen.split(",") if args.folizen != "all" else ["small", "medium", "large"]):
+        c = synth.FOLIZEN_SHAPES[name]
+        n_layers = args.folizen_layers or c["layers"]
+        n_prompt, n_ctx = args.folizen_prompt, min(c["window"] + 256, 4352)
+        toks = rng.integers(0, c["vocab"], n_prompt).astype(np.uint32)
+        arms = ["folizen", "llama"] if args.folizen_arm == "both" else [args.folizen_arm]
+        entry = {"shape": name, "layers": n_layers, **{k: c[k] for k in ("hidden", "heads", "kv_heads", "dim", "window", "ff", "vocab")}}
+        for arm in arms:
+            if arm == "folizen":
+                eng = k2.Engine(ctx, synth.random_folizen(name, seed=3, max_seq=n_ctx + 4 * steps + n_prompt, layers=n_layers))
+            else:
+                lc = dict(hidden=c["hidden"], layers=n_layers, n_q=c["heads"], n_kv=c["kv_heads"], head_dim=c["dim"], inter=c["ff"], vocab=c["vocab"],
+                          max_seq=n_ctx + 4 * steps + n_prompt, eps=1e-6, theta=1e6)
+                eng = k2.Engine(ctx, synth.random_model(lc, "nf4g128", seed=5, untied=True, share_layers=True))
+            eng.forward_token_ids(toks)                                   # warm-up: kernels loaded
+            l0 = ctx.launch_count
+            ms_p = timed(lambda: eng.forward_token_ids(toks), args.folizen_reps)
+            launches_prompt = (ctx.launch_count - l0) // args.folizen_reps
+            pos = 0
+            while pos < n_ctx:
+                n = min(n_ctx - pos, n_prompt)
+                eng.forward_token_ids(toks[:n], pos_start=pos)
+                pos += n
+            eng.decode_greedy(1, pos, 3)
+            pos += 3
+            best = None
+            for _ in range(args.folizen_reps):
+                ms = timed(lambda: eng.decode_greedy(1, pos, steps), 1)
+                pos += steps
+                best = ms if best is None else min(best, ms)
+            tok_s = steps / (best / 1e3)
+            res = {"prompt_tokens": n_prompt, "prompt_tok_s": round(n_prompt / (ms_p / 1e3)), "prompt_launches": int(launches_prompt), "decode_ctx": n_ctx,
+                   "decode_tok_s": round(tok_s, 1), "ms_per_token": round(best / steps, 4)}
+            if arm == "folizen":
+                wb, sb = _folizen_bytes(c, n_layers, n_ctx)
+                fl = _folizen_flops(c, n_layers)
+                res.update(bytes_per_token=wb + sb, decode_frac_of_copy_peak=round((wb + sb) * tok_s / 1e9 / peak, 4),
+                           prompt_tflops=round(fl * n_prompt / ms_p / 1e9, 1), prompt_frac_of_bf16_sustained=round(fl * n_prompt / ms_p / 1e9 / tf_peak, 4))
+            else:
+                per = eng.weight_bytes + eng.kv_bytes_per_pos * n_ctx
+                ops = _matmul_ops_per_token(dict(lc))
+                res.update(bytes_per_token=per, decode_frac_of_copy_peak=round(per * tok_s / 1e9 / peak, 4), prompt_int8_TOPs=round(ops * n_prompt / ms_p / 1e9, 1),
+                           prompt_frac_of_nominal_int8=round(ops * n_prompt / ms_p / 1e9 / 4500.0, 4))
+            if args.folizen_table:
+                res["step_table"] = eng.profile_step(1, pos, 8).splitlines()
+            entry[arm] = res
+            eng.close()
+        out["models"].append(entry)
+    out["clocks"] = sampler.stop()
+    print(json.dumps(out))
+    ctx.close()
+
+
 def cpu_decode_baseline():
     """The oracle's dense decode step on the same model shape, all host threads: 16 prompt tokens, 16 greedy steps."""
     sys.path.insert(0, os.path.join(ROOT, "oracle"))
@@ -992,6 +1096,13 @@ def main():
     ap.add_argument("--decode-ctx", type=int, default=15, help="--decode-only: position of the first greedy step")
     ap.add_argument("--kv-bits", type=int, default=8, choices=[4, 8], help="--decode-only: KV cache format")
     ap.add_argument("--split-kv", action="store_true", help="--decode-only: split-KV attention beyond 512 positions (the engine's opt-in flag)")
+    ap.add_argument("--folizen", default=None, metavar="SIZES", help="block models: small,medium,large or all - prompt and decode throughput beside a Llama shape of equal size")
+    ap.add_argument("--folizen-arm", default="both", choices=["both", "folizen", "llama"])
+    ap.add_argument("--folizen-layers", type=int, default=0, help="fewer layers than the shape's (profiling)")
+    ap.add_argument("--folizen-prompt", type=int, default=2048)
+    ap.add_argument("--folizen-steps", type=int, default=64)
+    ap.add_argument("--folizen-reps", type=int, default=3)
+    ap.add_argument("--folizen-table", action="store_true", help="add the per-kernel table of one decode step")
     ap.add_argument("--case", default=None, help="profile one case, e.g. b4:2048x49152 (fmt:KxN)")
     ap.add_argument("--tokens", type=int, default=1, help="tokens per launch in --case mode (1..4)")
     ap.add_argument("--no-graph", action="store_true", help="--case mode: skip the CUDA-graph replay timing")
@@ -1001,6 +1112,8 @@ def main():
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
     if args.decode_only or args.prefill_only:
         run_decode_only(args, local_rank)
+    elif args.folizen:
+        run_folizen(args, local_rank)
     elif args.case:
         run_case(args, local_rank)
     elif args.impl == "reference":

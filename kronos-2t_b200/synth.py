@@ -167,3 +167,35 @@ def random_model(cfg, mode, seed=0, modes=None, qkv_bias=False, untied=False, tp
     return dict(cfg=c, layers=layers, final_norm=np.ones(h, np.float32),
                 lm_head=random_matrix(seed * 100003 + 7 + 1000003 * tp_rank, c["vocab"], h, md["head"]),
                 rope=rope_table(c["max_seq"], hd, c["theta"]), embed_bf16=embed)
+
+
+# Block models (ffi.Engine specs with `blocks`) beside which a Llama shape of the same width, depth, heads and MLP makes sense
+FOLIZEN_SHAPES = {
+    "small": dict(hidden=1024, layers=12, heads=16, kv_heads=4, dim=64, window=1024, ff=4096, side_dim=32, rank=32, vocab=32768),
+    "medium": dict(hidden=2048, layers=24, heads=16, kv_heads=4, dim=128, window=2048, ff=8192, side_dim=64, rank=64, vocab=49152),
+    "large": dict(hidden=4096, layers=16, heads=32, kv_heads=8, dim=128, window=4096, ff=14336, side_dim=64, rank=96, vocab=131072),
+}
+
+
+def random_folizen(shape, seed=0, max_seq=8192, layers=None):
+    """Engine spec of a block model with random bf16 weights: attention with feed-forward and delta-rule blocks by turns.  Blocks
+    of a kind point at the same host arrays (each still becomes its own device copy)."""
+    c = dict(FOLIZEN_SHAPES[shape] if isinstance(shape, str) else shape)
+    n = layers or c["layers"]
+    h, H, G, d, ff, side = c["hidden"], c["heads"], c["kv_heads"], c["dim"], c["ff"], c["side_dim"]
+    rng = _rng(seed)
+
+    def mat(rows, cols):
+        base = int(np.float32(cols ** -0.5).view(np.uint32) >> 16) & 0x7F80      # magnitudes around 1 / sqrt(cols)
+        blk = rng.integers(base - 0x80, base + 0x80, min(rows * cols, 1 << 22), dtype=np.uint16) | (rng.integers(0, 2, min(rows * cols, 1 << 22), dtype=np.uint16) << 15)
+        return np.resize(blk, rows * cols).reshape(rows, cols)
+
+    one = lambda k: np.ones(k, np.float32)
+    tail = dict(norm1=one(h), side_norm=one(h) * 0.5, side_gate=mat(side, h), side_proj=mat(h, side))
+    attn = dict(tail, mixer=1, heads=H, kv_heads=G, dim=d, vdim=d, window=c["window"], ff=ff, q_norm=one(d), k_norm=one(d), head_scale=one(H) * d ** -0.5,
+                head_slope=(2.0 ** (-8.0 * (np.arange(H) + 1) / H)).astype(np.float32), in_proj=mat((H + 2 * G) * d, h), o_proj=mat(h, H * d), norm2=one(h),
+                act_coef=np.array([0.5, 0.3, 0.2, 0.0], np.float32), up_proj=mat(ff, h), down_proj=mat(h, ff))
+    delta = dict(tail, mixer=2, heads=H, dim=d, decay_rank=c["rank"], decay_scale=0.6065307, unit_eps=1e-6, decay_bias=-2.0 * one(H * d), rate_bias=-1.0 * one(H * d),
+                 out_norm=one(H * d), in_proj=mat(5 * H * d + c["rank"], h), decay_proj=mat(H * d, c["rank"]), o_proj=mat(h, H * d))
+    return dict(cfg=dict(hidden=h, vocab=c["vocab"], max_seq=max_seq, eps=1e-6, side_dim=side, precision=16), blocks=[attn if i % 2 == 0 else delta for i in range(n)],
+                final_norm=one(h), head=mat(c["vocab"], h), embed=mat(c["vocab"], h), side_embed=mat(c["vocab"], side * n))

@@ -132,13 +132,14 @@ def pointer_model(window, dtype_seed=0):
     t = model["tensors"]
     rng = np.random.default_rng(5)
     dirs = np.linalg.qr(rng.standard_normal((96, 3)))[0].T
+    t["embed"][:] = fm.bf16(t["embed"] - t["embed"] @ dirs[:2].T @ dirs[:2])          # the others have no part in the two directions
     t["embed"][1], t["embed"][2] = fm.bf16(30 * dirs[0]), fm.bf16(30 * dirs[1])
     for h in range(4):          # the same unit direction for the query of token 2 and the key of token 1
         u = np.sign(rng.standard_normal(32)) if h % 2 == 0 else u
-        t["l0.mix.q"][h * 32:(h + 1) * 32] = fm.bf16(0.02 * t["l0.mix.q"][h * 32:(h + 1) * 32] + np.outer(u, dirs[1]))
+        t["l0.mix.q"][h * 32:(h + 1) * 32] = fm.bf16(0.3 * t["l0.mix.q"][h * 32:(h + 1) * 32] + np.outer(u, dirs[1]))
         if h % 2 == 0:
             g = h // 2
-            t["l0.mix.k"][g * 32:(g + 1) * 32] = fm.bf16(0.02 * t["l0.mix.k"][g * 32:(g + 1) * 32] + np.outer(u, dirs[0]))
+            t["l0.mix.k"][g * 32:(g + 1) * 32] = fm.bf16(0.3 * t["l0.mix.k"][g * 32:(g + 1) * 32] + np.outer(u, dirs[0]))
     t["l0.mix.q.norm"][:] = t["l0.mix.k.norm"][:] = 1.0
     t["l0.mix.temp"][:] = [3.0, 3.0, 2.0, 2.0]
     return model
@@ -171,7 +172,7 @@ def test_window_edge(engine, window, how, dtype):
             other = json.loads(json.dumps(model["config"]))
             other["layers"][0]["mixer"]["mask"]["size"] = wrong
             bad, _ = ref.forward(dict(config=other, tensors=model["tensors"]), toks)
-            assert fm.error(bad, want)[-1] > 4 * TOL[dtype]
+            assert fm.error(bad, want)[-1] > 3 * TOL[dtype]
 
 
 def test_bias_and_temperature_show(engine):
