@@ -68,68 +68,99 @@ __global__ void __launch_bounds__(1024) block_norm_kernel(float *__restrict__ x,
 
 // A cluster of `cs` CTAs per token; CTA r holds the panels [r np / cs, (r + 1) np / cs) of the vector.  Three exchanges over
 // distributed shared memory: the sublayer's sum of squares, the partial gate products, the token input's sum of squares.
-// The CTA's share of both weight matrices is pulled towards L2 before the dependency wait.
+// The CTA's share of both weight matrices is bulk-copied to shared memory before the dependency wait (STAGED: bf16 panels that
+// fit), so after the wait only the two vectors come from global memory.
 constexpr uint32_t NS_THREADS = 256;
 constexpr uint32_t NS_MAX_CS = 8;
+constexpr uint32_t NS_WAIT_LIMIT = 1u << 22;
 
 __host__ __device__ inline uint32_t ns_slice_panels(uint32_t np, uint32_t cs) { return (np + cs - 1) / cs; }
-inline size_t ns_smem(uint32_t n, uint32_t dim, uint32_t cs) {
+inline size_t ns_vec_smem(uint32_t n, uint32_t dim, uint32_t cs) {
     const uint32_t slice = ns_slice_panels((n + 63) / 64, cs) * 64, dp = (dim + 63) / 64 * 64;
-    return ((size_t)2 * slice + (size_t)cs * dim + 2 * dp) * 4;
+    return (((size_t)2 * slice + dp + (size_t)cs * dim) * 4 + 127) & ~(size_t)127;
+}
+inline size_t ns_weight_smem(uint32_t n, uint32_t dim, uint32_t cs) {
+    const uint32_t sp = ns_slice_panels((n + 63) / 64, cs), dp = (dim + 63) / 64;
+    return (size_t)sp * dim * 128 + (size_t)dp * sp * 64 * 128;
 }
 
-template <bool F32>
+template <bool F32, bool STAGED>
 __global__ void __launch_bounds__(NS_THREADS) norm_side_kernel(float *__restrict__ x, size_t x_stride, const float *__restrict__ y, size_t y_stride, const float *__restrict__ w,
-                                                              uint32_t n, float eps, const SideArgs sd, const Act out) {
-    extern __shared__ __align__(16) float sm[];
+                                                              uint32_t n, float eps, const SideArgs sd, const Act out, uint32_t weights_at, uint32_t *__restrict__ err_flag) {
+    extern __shared__ __align__(128) float sm[];
     __shared__ float scratch[32], slot_a[NS_MAX_CS], slot_b[NS_MAX_CS];
+    __shared__ __align__(8) uint64_t bar_w;
     const uint32_t cs = cluster_size(), me = cluster_rank(), t = blockIdx.x / cs, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const uint32_t np = (n + 63) / 64, p0 = min(np, me * ns_slice_panels(np, cs)), p1 = min(np, p0 + ns_slice_panels(np, cs));
-    const uint32_t slice = ns_slice_panels(np, cs) * 64, dim = sd.dim, dp = (dim + 63) / 64 * 64;
-    float *s_x = sm, *s_y = s_x + slice, *s_g = s_y + slice, *s_part = s_g + 2 * dp;      // s_part [cs][dim]: written by the peers
+    const uint32_t np = (n + 63) / 64, sp = ns_slice_panels(np, cs), p0 = min(np, me * sp), p1 = min(np, p0 + sp);
+    const uint32_t slice = sp * 64, dim = sd.dim, dp = (dim + 63) / 64 * 64;
+    float *s_x = sm, *s_y = s_x + slice, *s_g = s_y + slice, *s_part = s_g + dp;      // s_part [cs][dim]: written by the peers
     const uint32_t k0 = p0 * 64, k1 = min(n, p1 * 64);
-    if (!F32) {
-        const char *gb = static_cast<const char *>(sd.gate.base), *pb = static_cast<const char *>(sd.proj.base);
-        for (uint32_t i = tid; i < (p1 - p0) * dim; i += NS_THREADS)
-            asm volatile("prefetch.global.L2 [%0];" ::"l"(gb + ((size_t)(p0 + i / dim) * sd.gate.rows_pad + i % dim) * 128));
-        const uint32_t rows = k1 > k0 ? k1 - k0 : 0;
-        for (uint32_t i = tid; i < rows * sd.proj.panels; i += NS_THREADS)
-            asm volatile("prefetch.global.L2 [%0];" ::"l"(pb + ((size_t)(i / rows) * sd.proj.rows_pad + k0 + i % rows) * 128));
+    DenseView gate = sd.gate, proj = sd.proj;
+    const uint32_t bar = (uint32_t)__cvta_generic_to_shared(&bar_w);
+    if (STAGED) {
+        uint8_t *s_w = reinterpret_cast<uint8_t *>(sm) + weights_at;
+        const uint32_t mine = p1 - p0, sw = (uint32_t)__cvta_generic_to_shared(s_w);
+        if (tid == 0) {
+            mbar_init(bar, 1);
+            fence_mbar_init();
+            mbar_expect_tx(bar, mine * dim * 128 + proj.panels * mine * 64 * 128);
+            const uint8_t *gb = static_cast<const uint8_t *>(sd.gate.base), *pb = static_cast<const uint8_t *>(sd.proj.base);
+            for (uint32_t p = 0; p < mine; ++p) bulk_g2s(sw + p * dim * 128, gb + (size_t)(p0 + p) * sd.gate.rows_pad * 128, dim * 128, bar);
+            for (uint32_t q = 0; q < proj.panels && mine > 0; ++q)
+                bulk_g2s(sw + mine * dim * 128 + q * mine * 64 * 128, pb + ((size_t)q * sd.proj.rows_pad + k0) * 128, mine * 64 * 128, bar);
+        }
+        gate.base = s_w; gate.rows_pad = dim;
+        proj.base = s_w + mine * dim * 128; proj.rows_pad = mine * 64;
     }
     for (uint32_t i = tid; i < slice; i += NS_THREADS) s_x[i] = 0.0f;
     for (uint32_t i = tid; i < dp; i += NS_THREADS) s_g[i] = 0.0f;
     pdl_wait();
     pdl_trigger();
-    cluster_sync_all();                         // every CTA of the cluster runs before its shared memory is written from outside
+    if (cs > 1) cluster_sync_all();             // every CTA of the cluster runs before its shared memory is written from outside
     float *xr = x + t * x_stride;
     const float *yr = y + t * y_stride;
+    const uint16_t *e = sd.table + (size_t)__ldcg(sd.tokens + t) * sd.table_stride + sd.offset;
+    const float e_first = tid < dim ? bf16_bits_to_f32(__ldg(e + tid)) : 0.0f;
     // sublayer output: x + y / rms(y) * w
     float ss[1] = {0.0f};
-    for (uint32_t k = k0 + tid; k < k1; k += NS_THREADS) { const float v = __ldcg(yr + k); s_y[k - k0] = v; ss[0] = __fmaf_rn(v, v, ss[0]); }
+    for (uint32_t k = k0 + tid; k < k1; k += NS_THREADS) {
+        const float v = __ldcg(yr + k);
+        s_x[k - k0] = __ldcg(xr + k);
+        s_y[k - k0] = v;
+        ss[0] = __fmaf_rn(v, v, ss[0]);
+    }
     block_sum<1>(ss, scratch);
     cluster_sum<1>(ss, slot_a);
     const float inv = 1.0f / sqrtf(ss[0] / (float)n + eps);
-    for (uint32_t k = k0 + tid; k < k1; k += NS_THREADS) s_x[k - k0] = __ldcg(xr + k) + s_y[k - k0] * inv * __ldg(w + k);
+    for (uint32_t k = k0 + tid; k < k1; k += NS_THREADS) s_x[k - k0] += s_y[k - k0] * inv * __ldg(w + k);
+    if (STAGED) {
+        bool ok = false;
+        for (uint32_t spin = 0; spin < NS_WAIT_LIMIT && !ok; ++spin) ok = mbar_try_wait(bar, 0u);
+        if (!ok && err_flag != nullptr) atomicExch(err_flag, 1u);
+    }
     __syncthreads();
     // partial gate products of the slice: eight lanes per row, four rows per warp and step
-    const uint32_t sub = lane & 7u;
+    const uint32_t sub = lane & 7u, q0 = STAGED ? 0u : p0, q1 = STAGED ? p1 - p0 : p1;
+#pragma unroll 2
     for (uint32_t r0 = warp * 4; r0 < dim; r0 += NS_THREADS / 8) {
         const uint32_t r = r0 + (lane >> 3);
-        const float d = row_dot8<F32>(sd.gate, min(r, dim - 1), p0, p1, s_x, sub);
+        const float d = row_dot8<F32, STAGED>(gate, min(r, dim - 1), q0, q1, s_x, sub);
         if (r < dim && sub < cs) st_cluster_f32(s_part + (size_t)me * dim + r, sub, d);
     }
-    cluster_sync_all();
-    const uint16_t *e = sd.table + (size_t)__ldcg(sd.tokens + t) * sd.table_stride + sd.offset;
+    if (cs > 1) cluster_sync_all();
+    else __syncthreads();
     for (uint32_t i = tid; i < dim; i += NS_THREADS) {
         float z = 0.0f;
         for (uint32_t r = 0; r < cs; ++r) z = __fadd_rn(z, s_part[(size_t)r * dim + i]);
-        s_g[i] = gelu_tanh(z) * bf16_bits_to_f32(__ldg(e + i));
+        s_g[i] = gelu_tanh(z) * (i == tid ? e_first : bf16_bits_to_f32(__ldg(e + i)));
     }
     __syncthreads();
     float s2[1] = {0.0f};
+    const uint32_t row_off = STAGED ? k0 : 0u;
+#pragma unroll 4
     for (uint32_t r0 = k0 + warp * 4; r0 < k1; r0 += NS_THREADS / 8) {
         const uint32_t r = r0 + (lane >> 3);
-        const float d = row_dot8<F32>(sd.proj, min(r, k1 - 1), 0, sd.proj.panels, s_g, sub);
+        const float d = row_dot8<F32, STAGED>(proj, min(r, k1 - 1) - row_off, 0, proj.panels, s_g, sub);
         if (r < k1 && sub == 0) { s_y[r - k0] = d; s2[0] = __fmaf_rn(d, d, s2[0]); }
     }
     block_sum<1>(s2, scratch);
@@ -214,16 +245,18 @@ cudaError_t launch_block_norm(cudaStream_t s, bool f32, bool add, float *x, size
     return launch_kernel(k, dim3(n_tok), dim3(threads), 0, s, pdl, x, x_stride, y, y_stride, w, n, eps, out);
 }
 
-bool norm_side_fits(uint32_t n, uint32_t dim) { return ns_smem(n, dim, 1) <= 200 * 1024; }
+bool norm_side_fits(uint32_t n, uint32_t dim) { return ns_vec_smem(n, dim, 1) <= 200 * 1024; }
 
 cudaError_t launch_norm_side(cudaStream_t s, bool f32, float *x, size_t x_stride, const float *y, size_t y_stride, const float *w, uint32_t n, float eps,
-                             const SideArgs &side, const Act &out, uint32_t n_tok, bool pdl) {
+                             const SideArgs &side, const Act &out, uint32_t n_tok, uint32_t *err_flag, bool pdl) {
     const uint32_t cs = cluster_for((n + 63) / 64, n_tok);
-    const size_t smem = ns_smem(n, side.dim, cs);
-    auto k = f32 ? norm_side_kernel<true> : norm_side_kernel<false>;
+    const size_t vec = ns_vec_smem(n, side.dim, cs), all = vec + ns_weight_smem(n, side.dim, cs);
+    const bool staged = !f32 && all <= 200 * 1024;
+    auto k = f32 ? norm_side_kernel<true, false> : staged ? norm_side_kernel<false, true> : norm_side_kernel<false, false>;
+    const size_t smem = staged ? all : vec;
     cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(k), smem);
     if (e != cudaSuccess) return e;
-    return launch_cluster(k, dim3(cs * n_tok), dim3(NS_THREADS), smem, s, pdl, cs, x, x_stride, y, y_stride, w, n, eps, side, out);
+    return launch_cluster(k, dim3(cs * n_tok), dim3(NS_THREADS), smem, s, pdl, cs, x, x_stride, y, y_stride, w, n, eps, side, out, (uint32_t)vec, err_flag);
 }
 
 cudaError_t launch_side_gelu(cudaStream_t s, bool f32, const float *z, size_t z_stride, const SideArgs &side, const Act &out, uint32_t n_tok, bool pdl) {

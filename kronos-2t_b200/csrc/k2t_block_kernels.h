@@ -24,7 +24,7 @@ struct SideArgs {
 };
 // short batches: residual add of the sublayer output y, and the token input, in one launch (a thread-block cluster per token)
 cudaError_t launch_norm_side(cudaStream_t s, bool f32, float *x, size_t x_stride, const float *y, size_t y_stride, const float *w, uint32_t n, float eps,
-                             const SideArgs &side, const Act &out, uint32_t n_tok, bool pdl);
+                             const SideArgs &side, const Act &out, uint32_t n_tok, uint32_t *err_flag, bool pdl);
 bool norm_side_fits(uint32_t n, uint32_t dim);
 // prompt batches: z [n_tok][dim] = gate x is a dense product; this makes the activation of `proj`
 cudaError_t launch_side_gelu(cudaStream_t s, bool f32, const float *z, size_t z_stride, const SideArgs &side, const Act &out, uint32_t n_tok, bool pdl);
@@ -45,6 +45,7 @@ struct WindowAttnArgs {
     float eps;
     Act out;                           // [n_tok][n_q * vdim]
 };
+bool window_attn_fits(bool f32, uint32_t group, uint32_t row);       // queries of a group beside one another in shared memory
 uint32_t window_attn_row(uint32_t dim, uint32_t vdim);       // cache row in elements; 0 = larger than the kernels support
 // n_tok == 1: one kernel (norms, cache row, attention); prompts: cache rows and queries, then the attention.  Returns the launches.
 cudaError_t launch_window_attention(cudaStream_t s, bool f32, const WindowAttnArgs &a, uint32_t n_tok, int sm_count, uint32_t *launches, bool pdl);
@@ -58,13 +59,14 @@ struct DeltaArgs {
     float *state;
     const float *decay_logit;          // prompts: decay product [n_tok][logit_stride]
     size_t logit_stride;
-    float *rec, *o;                    // prompts, scratch: [heads][n_tok][6 drow], [n_tok][heads][drow]
+    float *rec, *o;                    // prompts, scratch: delta_record_floats(n_tok, ..), [n_tok][heads][drow]
     uint32_t heads, dim, drow, rank;
     float decay_scale, unit_eps, eps;
     Act out;                           // [n_tok][heads * dim]
     uint32_t *err_flag;
 };
-uint32_t delta_row(uint32_t dim);      // dim rounded up to 32; 0 = larger than the kernels support
+uint32_t delta_row(uint32_t dim);      // dim rounded up to 64; 0 = larger than the kernels support
+size_t delta_record_floats(uint32_t n_tok, uint32_t heads, uint32_t drow);
 bool delta_step_fits(const DeltaArgs &a);
 cudaError_t launch_delta_step(cudaStream_t s, bool f32, const DeltaArgs &a, bool pdl);                                   // one token, one launch
 cudaError_t launch_delta_tanh(cudaStream_t s, bool f32, const DeltaArgs &a, const Act &out, uint32_t n_tok, bool pdl);   // activation of the decay product

@@ -108,7 +108,7 @@ bool finish_block(KronosCudaEngine *e, size_t l, const float *w, const Act &ax, 
     const SideArgs sd = side_args(e, l);
     const uint32_t h = e->cfg.hidden_size;
     if (T <= 16 && norm_side_fits(h, b.side_dim))
-        return engine_count(e, launch_norm_side(s, b.f32, b.x, b.hs, b.proj, b.hs, w, h, e->cfg.rms_norm_eps, sd, ax, T, e->pdl), "residual norm + token input");
+        return engine_count(e, launch_norm_side(s, b.f32, b.x, b.hs, b.proj, b.hs, w, h, e->cfg.rms_norm_eps, sd, ax, T, e->ctx->d_err, e->pdl), "residual norm + token input");
     const Act as = act_of(b, b.act_s, T, b.side_dim);
     return norm_add(e, w, ax, T) && product(e, B.side_gate, ax, T, b.z, b.zs, "token input gate") &&
            engine_count(e, launch_side_gelu(s, b.f32, b.z, b.zs, sd, as, T, e->pdl), "token input gelu") &&
@@ -317,7 +317,8 @@ extern "C" KronosCudaEngine *kronos_cuda_engine_create_blocks(KronosCudaContext 
         if (d.mixer == KRONOS_CUDA_MIXER_WINDOW_ATTENTION) {
             if (B.kv_heads == 0 || B.heads % B.kv_heads || B.vdim == 0) return bad(at + "query heads must be a multiple of the key/value heads");
             B.row = window_attn_row(B.dim, B.vdim);
-            if (B.row == 0 || B.heads / B.kv_heads > 64) return bad(at + "attention: head sizes up to 256, up to 64 query heads per key/value head");
+            if (B.row == 0) return bad(at + "attention: head sizes up to 256");
+            if (!window_attn_fits(b->f32, B.heads / B.kv_heads, B.row)) return bad(at + "attention: too many query heads per key/value head for this head size");
             const uint32_t rows = B.heads * B.dim + B.kv_heads * (B.dim + B.vdim);
             mix_cols = B.heads * B.vdim;
             if (!vec(B.q_norm, d.q_norm, B.dim) || !vec(B.k_norm, d.k_norm, B.dim) || !vec(B.head_scale, d.head_scale, B.heads) || !vec(B.head_slope, d.head_slope, B.heads) ||
@@ -346,7 +347,7 @@ extern "C" KronosCudaEngine *kronos_cuda_engine_create_blocks(KronosCudaContext 
             z_cols = std::max(z_cols, rows);
             s_cols = std::max(s_cols, B.rank);
             logit_cols = std::max(logit_cols, hd);
-            rec_floats = std::max(rec_floats, (size_t)B.heads * 6 * B.row);
+            rec_floats = std::max(rec_floats, delta_record_floats(MB, B.heads, B.row));
             o_floats = std::max(o_floats, (size_t)B.heads * B.row);
         } else {
             return bad(at + "unknown mixer " + std::to_string(d.mixer));
@@ -368,7 +369,7 @@ extern "C" KronosCudaEngine *kronos_cuda_engine_create_blocks(KronosCudaContext 
     if (!upload(b->head, *head, c.vocab_size, h) || !vec(b->final_norm, final_norm, h) || !dev_alloc(e, b->embed, (size_t)c.vocab_size * h, embed_bf16) ||
         (side_embed_bf16 && !dev_alloc(e, b->side_embed, (size_t)c.vocab_size * c.side_dim * n_blocks, side_embed_bf16)) ||
         !dev_alloc(e, b->x, (size_t)MB * b->hs) || !dev_alloc(e, b->z, (size_t)MB * b->zs) || !dev_alloc(e, b->proj, (size_t)MB * b->hs) || !dev_alloc(e, b->logit, (size_t)MB * b->ls) ||
-        !dev_alloc(e, b->rec, (size_t)MB * rec_floats) || !dev_alloc(e, b->scan_o, (size_t)MB * o_floats) || !act(b->act_x, h) || !act(b->act_m, m_cols) || !act(b->act_s, s_cols) ||
+        !dev_alloc(e, b->rec, rec_floats) || !dev_alloc(e, b->scan_o, (size_t)MB * o_floats) || !act(b->act_x, h) || !act(b->act_m, m_cols) || !act(b->act_s, s_cols) ||
         !dev_alloc(e, q, (size_t)MB * q_elems * (bits / 8)) || !dev_alloc(e, e->logits, (size_t)MB * c.vocab_size) || !dev_alloc(e, e->d_token, MB) || !dev_alloc(e, e->d_pos, 1) ||
         !dev_alloc(e, e->d_step, 1) || !dev_alloc(e, e->d_history, c.max_seq_len) || !dev_alloc(e, e->d_dbg, 32) || !dev_alloc(e, e->argmax_scratch, ARGMAX_SCRATCH_WORDS) ||
         !cuda_ok(ctx, cudaStreamSynchronize(ctx->stream), "engine_create_blocks"))

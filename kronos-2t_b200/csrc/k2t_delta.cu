@@ -5,9 +5,9 @@
 //   * delta_step_kernel (one token): CTA = head.  The state is requested before the dependency wait (only the same layer's
 //     previous step wrote it), then coefficients, recurrence, per-head norm, output gate and the activation of the output
 //     projection in one launch.
-//   * prompts: delta_prep_kernel writes the coefficients of every (head, token) as one record, delta_scan_kernel walks the
-//     tokens - CTA = 16 columns of a head, warp = 4 columns, eight lanes share a column's keys - with the records streamed
-//     through a ring of bulk copies and packed fp32 pairs (fma.rn.f32x2), delta_post_kernel norms and gates.
+//   * prompts: delta_prep_kernel writes the coefficients of every head and group of four tokens as one record,
+//     delta_scan_kernel walks the groups - a warp holds four columns, its lanes share the keys - with the records streamed through
+//     a ring of bulk copies and packed fp32 pairs (fma.rn.f32x2), delta_post_kernel norms and gates.
 #include <algorithm>
 
 #include "k2t_block_kernels.h"
@@ -25,16 +25,11 @@ __device__ __forceinline__ float decay_minus_one(float scale, float logit) { ret
 __device__ __forceinline__ uint64_t pk(float a, float b) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
 __device__ __forceinline__ void upk(uint64_t v, float &a, float &b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
 __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) { uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
-__device__ __forceinline__ ulonglong2 lds2(uint32_t saddr) {
-    ulonglong2 v;
-    asm volatile("ld.shared.v2.u64 {%0, %1}, [%2];" : "=l"(v.x), "=l"(v.y) : "r"(saddr));
-    return v;
-}
 
 // ------------------------------------------------------------------------------------------------ one token
 // thread = (four columns, sixteen keys): drow^2 / 64 threads
 constexpr uint32_t ST_KEYS = 16;
-inline uint32_t step_threads(uint32_t drow) { return std::max(64u, drow / 4 * (drow / ST_KEYS)); }
+inline uint32_t step_threads(uint32_t drow) { return std::max(128u, drow / 4 * (drow / ST_KEYS)); }
 inline size_t step_smem(uint32_t drow, uint32_t rank_pad) { return ((size_t)drow * (6 + drow / ST_KEYS) + rank_pad) * 4; }
 
 template <bool F32>
@@ -52,6 +47,9 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
         for (uint32_t i = 0; i < ST_KEYS; ++i) st[i] = __ldcg(reinterpret_cast<const float4 *>(state + (size_t)i * D));
     for (uint32_t i = tid; i < 6 * D; i += nthr) sm[i] = 0.0f;
     for (uint32_t i = tid; i < rank_pad; i += nthr) s_t[i] = 0.0f;
+    if (!F32)           // the head's rows of the decay product: weights, fetched while the predecessor runs
+        for (uint32_t i = tid; i < dim * a.decay.panels; i += nthr)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(static_cast<const char *>(a.decay.base) + ((size_t)(i / dim) * a.decay.rows_pad + h * dim + i % dim) * 128));
     pdl_wait();
     pdl_trigger();
     __syncthreads();
@@ -69,6 +67,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
     block_sum<1>(kk, scratch);                          // its barriers also publish s_t, s_k
     const float inv_k = 1.0f / sqrtf(kk[0] + a.unit_eps);
     const uint32_t sub = lane & 7u;
+#pragma unroll 4
     for (uint32_t r0 = warp * 4; r0 < dim; r0 += nthr / 8) {
         const uint32_t i = r0 + (lane >> 3), ii = min(i, dim - 1), c = h * dim + ii;
         const float z = row_dot8<F32>(a.decay, c, 0, a.decay.panels, s_t, sub) + __ldg(a.decay_bias + c);
@@ -134,63 +133,126 @@ __global__ void __launch_bounds__(256) delta_tanh_kernel(const float *__restrict
     act_store<F32>(out, i / rank, i % rank, tanhf(__ldcg(in + (i / rank) * in_stride + i % rank)));
 }
 
-// one warp per (token, head): record [w - 1 | a u | u | k | r | v], drow floats each
+// Prompts run in groups of four tokens.  With S the state ahead of a group, the products c_t = u_t^T S_(t-1) the removals need are
+//   c_t = U_t^T S + sum over s < t of (G_ts v_s - H_ts c_s),   U_t = u_t w_0 .. w_(t-1),
+//   G_ts = (u_t w_(s+1) .. w_(t-1))^T k_s,   H_ts = (u_t w_(s+1) .. w_(t-1))^T (a u)_s   (products by key channel),
+// so the four reductions over the keys of a column go side by side and one round of shuffles serves four tokens.  A group's
+// record: four times [w - 1 | a u | U | k | r | v] of drow floats, then G and H of the pairs (1,0) (2,0) (2,1) (3,0) (3,1) (3,2).
+constexpr uint32_t GROUP = 4;
+__host__ __device__ constexpr uint32_t group_floats(uint32_t drow) { return GROUP * 6 * drow + 16; }
+
+template <int NI>       // drow = 32 NI; one warp per (group, head)
 __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a, uint32_t n_tok) {
-    const uint32_t lane = threadIdx.x & 31, h = blockIdx.y, t = blockIdx.x * 8 + (threadIdx.x >> 5), D = a.drow, dim = a.dim, HD = a.heads * dim;
+    constexpr uint32_t D = 32 * NI;
+    const uint32_t lane = threadIdx.x & 31, h = blockIdx.y, g = blockIdx.x * 8 + (threadIdx.x >> 5), dim = a.dim, HD = a.heads * dim, groups = (n_tok + GROUP - 1) / GROUP;
     pdl_wait();
     pdl_trigger();
-    if (t >= n_tok) return;
-    const float *in = a.in + t * a.in_stride + h * dim, *lg = a.decay_logit + t * a.logit_stride + h * dim;
-    float *rec = a.rec + ((size_t)h * n_tok + t) * 6 * D;
-    float kk = 0.0f;
-    for (uint32_t i = lane; i < dim; i += 32) { const float k = __ldcg(in + HD + i); kk = __fmaf_rn(k, k, kk); }
-    const float inv_k = 1.0f / sqrtf(warp_sum(kk) + a.unit_eps);
-    for (uint32_t i = lane; i < D; i += 32) {
-        float w = 0.0f, au = 0.0f, u = 0.0f, k = 0.0f, r = 0.0f, v = 0.0f;
-        if (i < dim) {
-            k = __ldcg(in + HD + i);
-            u = k * inv_k;
-            w = decay_minus_one(a.decay_scale, __ldcg(lg + i) + __ldg(a.decay_bias + h * dim + i));
-            au = sigmoidf(__ldcg(in + 4 * HD + i) + __ldg(a.rate_bias + h * dim + i)) * u;
-            r = __ldcg(in + i);
-            v = __ldcg(in + 2 * HD + i);
+    if (g >= groups) return;
+    float *rec = a.rec + ((size_t)h * groups + g) * group_floats(D);
+    float k[GROUP][NI], inv_k[GROUP], sums[12];
+#pragma unroll
+    for (uint32_t t = 0; t < GROUP; ++t) {
+        const uint32_t tok = g * GROUP + t;
+        const float *in = a.in + tok * a.in_stride + h * dim;
+        float kk = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const uint32_t c = lane + 32 * i;
+            k[t][i] = tok < n_tok && c < dim ? __ldcg(in + HD + c) : 0.0f;
+            kk = __fmaf_rn(k[t][i], k[t][i], kk);
         }
-        rec[i] = w; rec[D + i] = au; rec[2 * D + i] = u; rec[3 * D + i] = k; rec[4 * D + i] = r; rec[5 * D + i] = v;
+        inv_k[t] = 1.0f / sqrtf(warp_sum(kk) + a.unit_eps);
     }
+#pragma unroll
+    for (int j = 0; j < 12; ++j) sums[j] = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const uint32_t c = lane + 32 * i;
+        float w[GROUP], au[GROUP];
+#pragma unroll
+        for (uint32_t t = 0; t < GROUP; ++t) {
+            const uint32_t tok = g * GROUP + t;
+            const float *in = a.in + tok * a.in_stride + h * dim;
+            float d = 0.0f, r = 0.0f, v = 0.0f;
+            au[t] = 0.0f;
+            float u = k[t][i] * inv_k[t];
+            if (tok < n_tok && c < dim) {
+                d = decay_minus_one(a.decay_scale, __ldcg(a.decay_logit + tok * a.logit_stride + h * dim + c) + __ldg(a.decay_bias + h * dim + c));
+                au[t] = sigmoidf(__ldcg(in + 4 * HD + c) + __ldg(a.rate_bias + h * dim + c)) * u;
+                r = __ldcg(in + c);
+                v = __ldcg(in + 2 * HD + c);
+            }
+            w[t] = 1.0f + d;
+            // u w_(t-1) .. w_(s+1) against k_s and (a u)_s, s from t - 1 down
+#pragma unroll
+            for (int s = GROUP - 2; s >= 0; --s)
+                if (s < (int)t) {
+                    const int pair = (int)t * ((int)t - 1) / 2 + s;
+                    sums[pair] = __fmaf_rn(u, k[s][i], sums[pair]);
+                    sums[6 + pair] = __fmaf_rn(u, au[s], sums[6 + pair]);
+                    u *= w[s];
+                }
+            float *q = rec + t * 6 * D + c;
+            q[0] = d; q[D] = au[t]; q[2 * D] = u; q[3 * D] = k[t][i]; q[4 * D] = r; q[5 * D] = v;
+        }
+    }
+    float mine = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 12; ++j) {
+        const float v = warp_sum(sums[j]);
+        if ((int)lane == j) mine = v;
+    }
+    if (lane < 16) rec[GROUP * 6 * D + lane] = mine;
 }
 
-constexpr uint32_t SC_STAGES = 3, SC_FLOATS = 6144;        // ring: stages of SC_FLOATS floats (1024 / drow records)
+constexpr uint32_t SC_STAGES = 3, SC_COLS = 4;
 constexpr uint32_t SC_WAIT_LIMIT = 1u << 22;
+__host__ __device__ constexpr uint32_t stage_groups(uint32_t drow) { return drow >= 256 ? 1u : 256u / drow; }
 
-template <int KI>       // drow = 32 KI: lane kl of a column's eight holds keys 4 (8 i + kl) .. + 3, i < KI
+// Sixteen values per lane summed over the warp: lane l returns the sum of value l / 2 (the exchange halves the values per step).
+__device__ __forceinline__ float warp_sum16(float (&v)[16], uint32_t lane) {
+#pragma unroll
+    for (int w = 8; w > 0; w >>= 1)
+#pragma unroll
+        for (int i = 0; i < w; ++i) {
+            const bool up = (lane & (2 * w)) != 0;
+            const float give = up ? v[i] : v[i + w], keep = up ? v[i + w] : v[i];
+            v[i] = __fadd_rn(keep, __shfl_xor_sync(0xffffffffu, give, 2 * w));
+        }
+    return __fadd_rn(v[0], __shfl_xor_sync(0xffffffffu, v[0], 1));
+}
+
+// CTA = four warps, warp = four columns of a head; the 32 lanes share the keys: lane l holds the key pairs 2 (32 i + l), i < KP
+// (drow = 64 KP), so a record vector is read once per warp, 256 consecutive bytes per load.
+template <int KP>
 __global__ void __launch_bounds__(128) delta_scan_kernel(const float *__restrict__ rec, uint32_t n_tok, float *__restrict__ state, float *__restrict__ o, uint32_t heads,
                                                         uint32_t *__restrict__ err_flag) {
     extern __shared__ __align__(128) float ring[];
     __shared__ __align__(8) uint64_t bars[SC_STAGES];
-    constexpr uint32_t D = 32 * KI, TB = 1024 / D, REC = 6 * D;
-    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, kl = lane & 7u, col = blockIdx.x * 16 + warp * 4 + (lane >> 3);
+    constexpr uint32_t D = 64 * KP, GF = group_floats(D), SG = stage_groups(D), STAGE = SG * GF;
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, col = (blockIdx.x * 4 + warp) * SC_COLS;
     const uint32_t bar = (uint32_t)__cvta_generic_to_shared(bars), rb = (uint32_t)__cvta_generic_to_shared(ring);
-    const float *src = rec + (size_t)h * n_tok * REC;
-    const uint32_t chunks = (n_tok + TB - 1) / TB;
+    const uint32_t groups = (n_tok + GROUP - 1) / GROUP, chunks = (groups + SG - 1) / SG;
+    const float *src = rec + (size_t)h * groups * GF;
     if (tid == 0) {
         for (uint32_t i = 0; i < SC_STAGES; ++i) mbar_init(bar + 8 * i, 1);
         fence_mbar_init();
     }
     float *sp = state + (size_t)h * D * D + col;
-    uint64_t s[KI][2];
+    uint64_t s[SC_COLS][KP];
 #pragma unroll
-    for (int i = 0; i < KI; ++i) {
-        const uint32_t key = (i * 8 + kl) * 4;
-        s[i][0] = pk(__ldcg(sp + (size_t)key * D), __ldcg(sp + (size_t)(key + 1) * D));
-        s[i][1] = pk(__ldcg(sp + (size_t)(key + 2) * D), __ldcg(sp + (size_t)(key + 3) * D));
+    for (int i = 0; i < KP; ++i) {
+        const float *q = sp + (size_t)((i * 32 + lane) * 2) * D;
+        const float4 e = __ldcg(reinterpret_cast<const float4 *>(q)), f = __ldcg(reinterpret_cast<const float4 *>(q + D));
+        s[0][i] = pk(e.x, f.x); s[1][i] = pk(e.y, f.y); s[2][i] = pk(e.z, f.z); s[3][i] = pk(e.w, f.w);
     }
     pdl_wait();
     pdl_trigger();
     __syncthreads();
     auto request = [&](uint32_t c) {
-        const uint32_t n = min(TB, n_tok - c * TB);
-        mbar_expect_tx(bar + 8 * (c % SC_STAGES), n * REC * 4);
-        bulk_g2s(rb + (c % SC_STAGES) * SC_FLOATS * 4, src + (size_t)c * TB * REC, n * REC * 4, bar + 8 * (c % SC_STAGES));
+        const uint32_t bytes = min(SG, groups - c * SG) * GF * 4;
+        mbar_expect_tx(bar + 8 * (c % SC_STAGES), bytes);
+        bulk_g2s(rb + (c % SC_STAGES) * STAGE * 4, src + (size_t)c * STAGE, bytes, bar + 8 * (c % SC_STAGES));
     };
     if (tid == 0)
         for (uint32_t c = 0; c < min(SC_STAGES, chunks); ++c) request(c);
@@ -203,62 +265,71 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float *__restrict
                 for (uint32_t spin = 0; spin < SC_WAIT_LIMIT && !mbar_try_wait(bar + 8 * (d % SC_STAGES), (d / SC_STAGES) & 1u); ++spin) {}
             return;
         }
-        const uint32_t n = min(TB, n_tok - c * TB);
-        uint32_t at = rb + (c % SC_STAGES) * SC_FLOATS * 4;
-#pragma unroll 2
-        for (uint32_t t = 0; t < n; ++t, at += REC * 4) {
-            const uint32_t ak = at + kl * 16;
-            uint64_t d0 = 0, d1 = 0;
+        const uint32_t n = min(SG, groups - c * SG);
+        const float *at = ring + (c % SC_STAGES) * STAGE;
+#pragma unroll 1
+        for (uint32_t gi = 0; gi < n; ++gi, at += GF) {
+            const uint64_t *vec = reinterpret_cast<const uint64_t *>(at) + lane;
+            auto part = [&](uint32_t t, uint32_t which, int i) { return vec[(t * 6 + which) * (D / 2) + i * 32]; };
+            float d[GROUP * SC_COLS], v[GROUP * SC_COLS];
 #pragma unroll
-            for (int i = 0; i < KI; ++i) {
-                const ulonglong2 u = lds2(ak + 2 * D * 4 + i * 128);
-                d0 = fma2(u.x, s[i][0], d0);
-                d1 = fma2(u.y, s[i][1], d1);
-            }
-            float v;
-            asm volatile("ld.shared.f32 %0, [%1];" : "=f"(v) : "r"(at + (5 * D + col) * 4));
-            const uint64_t v2 = pk(v, v);
+            for (uint32_t t = 0; t < GROUP; ++t) {
+                uint64_t p[SC_COLS];
 #pragma unroll
-            for (int i = 0; i < KI; ++i) {          // w S + k v^T does not need the reduced product
-                const ulonglong2 w = lds2(ak + i * 128), k = lds2(ak + 3 * D * 4 + i * 128);
-                s[i][0] = fma2(w.x, s[i][0], fma2(k.x, v2, s[i][0]));
-                s[i][1] = fma2(w.y, s[i][1], fma2(k.y, v2, s[i][1]));
-            }
-            float e0, e1, e2, e3;
-            upk(d0, e0, e1);
-            upk(d1, e2, e3);
-            float cc = __fadd_rn(__fadd_rn(e0, e1), __fadd_rn(e2, e3));
-            cc = __fadd_rn(cc, __shfl_xor_sync(0xffffffffu, cc, 1));
-            cc = __fadd_rn(cc, __shfl_xor_sync(0xffffffffu, cc, 2));
-            cc = __fadd_rn(cc, __shfl_xor_sync(0xffffffffu, cc, 4));
-            const uint64_t c2 = pk(-cc, -cc);
-            uint64_t o0 = 0, o1 = 0;
+                for (int i = 0; i < KP; ++i) {
+                    const uint64_t u = part(t, 2, i);
 #pragma unroll
-            for (int i = 0; i < KI; ++i) {
-                const ulonglong2 au = lds2(ak + D * 4 + i * 128), r = lds2(ak + 4 * D * 4 + i * 128);
-                s[i][0] = fma2(au.x, c2, s[i][0]);
-                s[i][1] = fma2(au.y, c2, s[i][1]);
-                o0 = fma2(r.x, s[i][0], o0);
-                o1 = fma2(r.y, s[i][1], o1);
+                    for (int c2 = 0; c2 < (int)SC_COLS; ++c2) p[c2] = fma2(u, s[c2][i], i == 0 ? 0ull : p[c2]);
+                }
+                const float4 v4 = *reinterpret_cast<const float4 *>(at + (t * 6 + 5) * D + col);
+                v[t * 4] = v4.x; v[t * 4 + 1] = v4.y; v[t * 4 + 2] = v4.z; v[t * 4 + 3] = v4.w;
+#pragma unroll
+                for (int c2 = 0; c2 < (int)SC_COLS; ++c2) { float e0, e1; upk(p[c2], e0, e1); d[t * 4 + c2] = __fadd_rn(e0, e1); }
             }
-            upk(o0, e0, e1);
-            upk(o1, e2, e3);
-            float oo = __fadd_rn(__fadd_rn(e0, e1), __fadd_rn(e2, e3));
-            oo = __fadd_rn(oo, __shfl_xor_sync(0xffffffffu, oo, 1));
-            oo = __fadd_rn(oo, __shfl_xor_sync(0xffffffffu, oo, 2));
-            oo = __fadd_rn(oo, __shfl_xor_sync(0xffffffffu, oo, 4));
-            if (kl == 0) o[((size_t)(c * TB + t) * heads + h) * D + col] = oo;
+            const float dm = warp_sum16(d, lane);
+#pragma unroll
+            for (int i = 0; i < 16; ++i) d[i] = __shfl_sync(0xffffffffu, dm, 2 * i);
+            const float *gh = at + GROUP * 6 * D;
+#pragma unroll
+            for (uint32_t t = 1; t < GROUP; ++t)
+#pragma unroll
+                for (uint32_t q = 0; q < t; ++q) {
+                    const float g = gh[t * (t - 1) / 2 + q], hh = -gh[6 + t * (t - 1) / 2 + q];
+#pragma unroll
+                    for (int c2 = 0; c2 < (int)SC_COLS; ++c2) d[t * 4 + c2] = __fmaf_rn(hh, d[q * 4 + c2], __fmaf_rn(g, v[q * 4 + c2], d[t * 4 + c2]));
+                }
+            float oo[GROUP * SC_COLS];
+#pragma unroll
+            for (uint32_t t = 0; t < GROUP; ++t) {
+                uint64_t v2[SC_COLS], c2n[SC_COLS], p[SC_COLS];
+#pragma unroll
+                for (int c2 = 0; c2 < (int)SC_COLS; ++c2) { v2[c2] = pk(v[t * 4 + c2], v[t * 4 + c2]); c2n[c2] = pk(-d[t * 4 + c2], -d[t * 4 + c2]); }
+#pragma unroll
+                for (int i = 0; i < KP; ++i) {
+                    const uint64_t w = part(t, 0, i), au = part(t, 1, i), k = part(t, 3, i), r = part(t, 4, i);
+#pragma unroll
+                    for (int c2 = 0; c2 < (int)SC_COLS; ++c2) {
+                        s[c2][i] = fma2(au, c2n[c2], fma2(w, s[c2][i], fma2(k, v2[c2], s[c2][i])));
+                        p[c2] = fma2(r, s[c2][i], i == 0 ? 0ull : p[c2]);
+                    }
+                }
+#pragma unroll
+                for (int c2 = 0; c2 < (int)SC_COLS; ++c2) { float e0, e1; upk(p[c2], e0, e1); oo[t * 4 + c2] = __fadd_rn(e0, e1); }
+            }
+            const float om = warp_sum16(oo, lane);
+            const uint32_t tok = (c * SG + gi) * GROUP + (lane >> 3);
+            if ((lane & 1u) == 0 && tok < n_tok) o[((size_t)tok * heads + h) * D + col + ((lane >> 1) & 3u)] = om;
         }
         __syncthreads();                        // the stage is free
         if (tid == 0 && c + SC_STAGES < chunks) request(c + SC_STAGES);
     }
 #pragma unroll
-    for (int i = 0; i < KI; ++i) {
-        const uint32_t key = (i * 8 + kl) * 4;
-        float e0, e1, e2, e3;
-        upk(s[i][0], e0, e1);
-        upk(s[i][1], e2, e3);
-        sp[(size_t)key * D] = e0; sp[(size_t)(key + 1) * D] = e1; sp[(size_t)(key + 2) * D] = e2; sp[(size_t)(key + 3) * D] = e3;
+    for (int i = 0; i < KP; ++i) {
+        float *q = sp + (size_t)((i * 32 + lane) * 2) * D;
+        float4 e, f;
+        upk(s[0][i], e.x, f.x); upk(s[1][i], e.y, f.y); upk(s[2][i], e.z, f.z); upk(s[3][i], e.w, f.w);
+        *reinterpret_cast<float4 *>(q) = e;
+        *reinterpret_cast<float4 *>(q + D) = f;
     }
 }
 
@@ -275,16 +346,20 @@ __global__ void __launch_bounds__(256) delta_post_kernel(const DeltaArgs a, uint
     for (uint32_t j = lane; j < dim; j += 32) act_store<F32>(a.out, t, h * dim + j, __ldcg(o + j) * inv * __ldg(a.norm + h * dim + j) * sigmoidf(__ldcg(g + j)));
 }
 
-template <int KI> cudaError_t scan_ki(cudaStream_t s, const DeltaArgs &a, uint32_t n_tok, bool pdl) {
-    const size_t smem = SC_STAGES * SC_FLOATS * 4;
-    cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(delta_scan_kernel<KI>), smem);
+template <int KP> cudaError_t scan_kp(cudaStream_t s, const DeltaArgs &a, uint32_t n_tok, bool pdl) {
+    const uint32_t groups = (n_tok + GROUP - 1) / GROUP;
+    cudaError_t e = launch_kernel(delta_prep_kernel<2 * KP>, dim3((groups + 7) / 8, a.heads), dim3(256), 0, s, pdl, a, n_tok);
     if (e != cudaSuccess) return e;
-    return launch_kernel(delta_scan_kernel<KI>, dim3(2 * KI, a.heads), dim3(128), smem, s, pdl, a.rec, n_tok, a.state, a.o, a.heads, a.err_flag);
+    constexpr size_t smem = (size_t)SC_STAGES * stage_groups(64 * KP) * group_floats(64 * KP) * 4;
+    e = allow_dynamic_smem(reinterpret_cast<const void *>(delta_scan_kernel<KP>), smem);
+    if (e != cudaSuccess) return e;
+    return launch_kernel(delta_scan_kernel<KP>, dim3(64 * KP / (4 * SC_COLS), a.heads), dim3(128), smem, s, pdl, a.rec, n_tok, a.state, a.o, a.heads, a.err_flag);
 }
 
 }  // namespace
 
-uint32_t delta_row(uint32_t dim) { return dim <= 256 ? (dim + 31u) & ~31u : 0u; }
+uint32_t delta_row(uint32_t dim) { return dim <= 256 ? (dim + 63u) & ~63u : 0u; }
+size_t delta_record_floats(uint32_t n_tok, uint32_t heads, uint32_t drow) { return (size_t)((n_tok + GROUP - 1) / GROUP) * heads * group_floats(drow); }
 bool delta_step_fits(const DeltaArgs &a) { return a.drow <= 128 && step_smem(a.drow, (a.rank + 63) / 64 * 64) <= 200 * 1024; }
 
 cudaError_t launch_delta_step(cudaStream_t s, bool f32, const DeltaArgs &a, bool pdl) {
@@ -301,18 +376,13 @@ cudaError_t launch_delta_tanh(cudaStream_t s, bool f32, const DeltaArgs &a, cons
 }
 cudaError_t launch_delta_prompt(cudaStream_t s, bool f32, const DeltaArgs &a, uint32_t n_tok, bool pdl) {
     const dim3 grid((n_tok + 7) / 8, a.heads);
-    cudaError_t e = launch_kernel(delta_prep_kernel, grid, dim3(256), 0, s, pdl, a, n_tok);
-    if (e != cudaSuccess) return e;
-    switch (a.drow / 32) {
-        case 1: e = scan_ki<1>(s, a, n_tok, pdl); break;
-        case 2: e = scan_ki<2>(s, a, n_tok, pdl); break;
-        case 3: e = scan_ki<3>(s, a, n_tok, pdl); break;
-        case 4: e = scan_ki<4>(s, a, n_tok, pdl); break;
-        case 5: e = scan_ki<5>(s, a, n_tok, pdl); break;
-        case 6: e = scan_ki<6>(s, a, n_tok, pdl); break;
-        case 7: e = scan_ki<7>(s, a, n_tok, pdl); break;
-        case 8: e = scan_ki<8>(s, a, n_tok, pdl); break;
-        default: e = cudaErrorInvalidValue;
+    cudaError_t e = cudaErrorInvalidValue;
+    switch (a.drow / 64) {
+        case 1: e = scan_kp<1>(s, a, n_tok, pdl); break;
+        case 2: e = scan_kp<2>(s, a, n_tok, pdl); break;
+        case 3: e = scan_kp<3>(s, a, n_tok, pdl); break;
+        case 4: e = scan_kp<4>(s, a, n_tok, pdl); break;
+        default: break;
     }
     if (e != cudaSuccess) return e;
     return launch_kernel(f32 ? delta_post_kernel<true> : delta_post_kernel<false>, grid, dim3(256), 0, s, pdl, a, n_tok);

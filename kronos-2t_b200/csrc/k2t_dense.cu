@@ -13,11 +13,10 @@ namespace {
 // A warp owns a group of eight rows and, with wk = 1 .. 8 warps per group, every wk-th panel of it: 1 KiB of consecutive
 // weights per step.  Lane = (row pair r, r + 4; chunk c): both rows use the same eight activation values.  The first GV_PF
 // panels are requested before the dependency wait, so a launch whose warps hold few panels has its whole matrix in flight
-// while the predecessor still runs.
-constexpr uint32_t GV_PF = 4;
-
-template <int NT>
-__global__ void __launch_bounds__(256) dense_gemv_kernel(const uint4 *__restrict__ w, uint32_t rows, uint32_t rows_pad, uint32_t np, const uint4 *__restrict__ x,
+// while the predecessor still runs
+// (four with four CTAs per SM, six with two: more bytes in flight where the rows give only few CTAs).
+template <int NT, int GV_PF>
+__global__ void __launch_bounds__(256, NT == 1 && GV_PF == 4 ? 4 : 2) dense_gemv_kernel(const uint4 *__restrict__ w, uint32_t rows, uint32_t rows_pad, uint32_t np, const uint4 *__restrict__ x,
                                                         uint32_t ld, uint32_t t0, uint32_t n_tok, float *__restrict__ out, size_t out_stride, uint32_t wk_log2) {
     __shared__ float s_part[8][8][NT];
     const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, wk = 1u << wk_log2, c = lane & 7u, r = lane >> 3;
@@ -85,10 +84,19 @@ __global__ void __launch_bounds__(256) dense_gemv_kernel(const uint4 *__restrict
 template <int NT>
 cudaError_t gemv_nt(cudaStream_t s, const DenseView &m, const Act &x, uint32_t t0, uint32_t n_tok, float *out, size_t out_stride, int sm_count, bool pdl) {
     const uint32_t groups = (m.rows + 7) / 8;
-    uint32_t wl = 0;       // warps per row group: about 20 warps per SM, and no more than the panels
-    while (wl < 3 && (2u << wl) <= m.panels && (groups << wl) < 14u * (uint32_t)sm_count) ++wl;
-    const uint32_t per = 8u >> wl;
-    return launch_kernel(dense_gemv_kernel<NT>, dim3((groups + per - 1) / per), dim3(256), 0, s, pdl, static_cast<const uint4 *>(m.base), m.rows, m.rows_pad, m.panels,
+    // warps per row group: the fewest rounds of panels over the waves of the grid (a CTA beyond a full wave costs a whole round)
+    const uint32_t slots = (uint32_t)sm_count * (NT == 1 ? 4u : 2u);
+    uint32_t wl = 0;
+    float best = 1e30f;
+    for (uint32_t l = 0; l <= 3 && (1u << l) <= m.panels; ++l) {
+        const uint32_t ctas = (groups + (8u >> l) - 1) / (8u >> l), waves = (ctas + slots - 1) / slots, steps = (m.panels + (1u << l) - 1) >> l;
+        // a step's time grows with the warps that share an SM's bandwidth, and has a floor of its own
+        const float fill = (float)ctas / (float)(waves * slots), t = (float)waves * (3.0f + (float)steps * (0.35f + 0.65f * fill));
+        if (t < best) { best = t; wl = l; }
+    }
+    const uint32_t per = 8u >> wl, ctas = (groups + per - 1) / per;
+    auto k = NT == 1 && ctas <= 2u * (uint32_t)sm_count ? dense_gemv_kernel<NT, NT == 1 ? 6 : 4> : dense_gemv_kernel<NT, 4>;
+    return launch_kernel(k, dim3(ctas), dim3(256), 0, s, pdl, static_cast<const uint4 *>(m.base), m.rows, m.rows_pad, m.panels,
                          static_cast<const uint4 *>(x.p), x.ld, t0, n_tok, out, out_stride, wl);
 }
 

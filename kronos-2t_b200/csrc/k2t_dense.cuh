@@ -40,8 +40,9 @@ __device__ __forceinline__ float dot8(const uint4 &w, const float *x, float acc)
     return acc;
 }
 // Product of matrix row `row`, panels [p0, p1), with x (shared memory; x[0] belongs to column 64 p0, zero beyond the last
-// column) by eight consecutive lanes (sub = lane % 8); every one of them receives the sum.
-template <bool F32> __device__ __forceinline__ float row_dot8(const DenseView &m, uint32_t row, uint32_t p0, uint32_t p1, const float *x, uint32_t sub) {
+// column) by eight consecutive lanes (sub = lane % 8); every one of them receives the sum.  SHARED: the panels were copied to
+// shared memory.
+template <bool F32, bool SHARED = false> __device__ __forceinline__ float row_dot8(const DenseView &m, uint32_t row, uint32_t p0, uint32_t p1, const float *x, uint32_t sub) {
     float acc = 0.0f;
     if (F32) {
         const float *w = static_cast<const float *>(m.base) + (size_t)row * m.rows_pad;
@@ -49,8 +50,11 @@ template <bool F32> __device__ __forceinline__ float row_dot8(const DenseView &m
         for (uint32_t k = p0 * PANEL + sub; k < k1; k += 8) acc = __fmaf_rn(__ldg(w + k), x[k - p0 * PANEL], acc);
     } else {
         const uint4 *w = static_cast<const uint4 *>(m.base);
-        for (uint32_t p = p0; p < p1; ++p)
-            acc = dot8(__ldg(w + ((size_t)p * m.rows_pad + row) * 8 + (sub ^ (row & 7u))), x + (p - p0) * PANEL + sub * 8, acc);
+#pragma unroll 4
+        for (uint32_t p = p0; p < p1; ++p) {
+            const uint4 *q = w + ((size_t)p * m.rows_pad + row) * 8 + (sub ^ (row & 7u));
+            acc = dot8(SHARED ? *q : __ldg(q), x + (p - p0) * PANEL + sub * 8, acc);
+        }
     }
     acc = __fadd_rn(acc, __shfl_xor_sync(0xffffffffu, acc, 1));
     acc = __fadd_rn(acc, __shfl_xor_sync(0xffffffffu, acc, 2));

@@ -79,23 +79,42 @@ __global__ void __launch_bounds__(256) window_prep_kernel(const AttnParams p) {
 }
 
 // ------------------------------------------------------------------------------------------------ one token per cluster
-constexpr uint32_t RW_THREADS = 256, RW_SC = 256, RW_HB = 8, RW_PB = 4;
-inline size_t rw_smem(uint32_t group, uint32_t row) { return ((size_t)group * (2 * row + RW_SC + 4) + 8 * RW_THREADS) * 4; }
+// The heads of a group run in passes of HB (the group is padded to full passes with zero queries), so the inner loops carry no
+// branches and a step's row loads are all in flight together.  A decode step pulls the cached rows it will read towards L2 before
+// its dependency wait: they were written by earlier steps, only the new row depends on the predecessor.
+constexpr uint32_t RW_THREADS = 256, RW_SC = 256, RW_MAX_CS = 8;
+__host__ __device__ inline uint32_t rw_pad(uint32_t group, uint32_t hb) { return (group + hb - 1) / hb * hb; }
+inline size_t rw_smem(uint32_t group, uint32_t row, uint32_t hb) {
+    return ((size_t)rw_pad(group, hb) * (2 * row + RW_SC + 4 + 2 * RW_MAX_CS) + (size_t)8 * RW_THREADS * hb) * 4;
+}
 
-template <typename T, int D>
+template <typename T, int D, int HB>
 __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams p) {
     extern __shared__ __align__(16) float sm[];
     const WindowAttnArgs &a = p.a;
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, cs = cluster_size(), me = cluster_rank();
-    const uint32_t g = blockIdx.y, t = blockIdx.z, group = a.n_q / a.n_kv;
-    float *s_q = sm, *s_o = s_q + group * D, *s_p = s_o + group * D, *s_m = s_p + group * RW_SC, *s_l = s_m + group, *s_al = s_l + group, *s_red = s_al + 2 * group;
-    pdl_wait();
-    pdl_trigger();
-    const uint32_t pos = __ldcg(a.pos) + t;
+    const uint32_t g = blockIdx.y, t = blockIdx.z, group = a.n_q / a.n_kv, gp = rw_pad(group, HB);
+    float *s_q = sm, *s_o = s_q + gp * D, *s_p = s_o + gp * D, *s_red = s_p + gp * RW_SC, *s_m = s_red + 8 * RW_THREADS * HB, *s_l = s_m + gp, *s_al = s_l + gp,
+          *s_fm = s_al + 2 * gp, *s_fl = s_fm + gp * RW_MAX_CS;
+    T *kc = static_cast<T *>(a.k_cache) + (size_t)g * p.ring_rows * D, *vc = static_cast<T *>(a.v_cache) + (size_t)g * p.ring_rows * D;
+    if (!p.fused) { pdl_wait(); pdl_trigger(); }
+    const uint32_t pos = __ldcg(a.pos) + t;                                              // a decode step's position was set before the step began
     const uint32_t n_seen = a.ring.active_len(pos + 1), lo = pos + 1 - n_seen;          // sinks are 0: the seen positions are consecutive
     const uint32_t per = (n_seen + cs - 1) / cs, j_lo = lo + min(n_seen, me * per), j_hi = lo + min(n_seen, (me + 1) * per);
-    T *kc = static_cast<T *>(a.k_cache) + (size_t)g * p.ring_rows * D, *vc = static_cast<T *>(a.v_cache) + (size_t)g * p.ring_rows * D;
     if (p.fused) {
+        constexpr uint32_t LINES = D * sizeof(T) / 64;
+        for (uint32_t i = tid; i < (j_hi - j_lo) * LINES; i += RW_THREADS) {
+            const size_t at = (size_t)a.ring.slot_of_pos(j_lo + i / LINES) * D * sizeof(T) + (i % LINES) * 64;
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(kc) + at));
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(vc) + at));
+        }
+    }
+    for (uint32_t i = tid; i < gp * D; i += RW_THREADS) s_o[i] = 0.0f;
+    for (uint32_t i = group * D + tid; i < gp * D; i += RW_THREADS) s_q[i] = 0.0f;
+    for (uint32_t i = tid; i < gp; i += RW_THREADS) { s_m[i] = -INFINITY; s_l[i] = 0.0f; s_al[i] = 0.0f; }
+    if (p.fused) {
+        pdl_wait();
+        pdl_trigger();
         const float *x = a.qkv + t * a.qkv_stride;
         for (uint32_t h = warp; h < group; h += RW_THREADS / 32) norm_row<float>(x + (g * group + h) * a.dim, a.q_norm, a.dim, D, a.eps, s_q + h * D, lane);
         if (pos >= j_lo && pos < j_hi) {            // the CTA that attends to the new position stores its rows
@@ -112,20 +131,20 @@ __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams
             for (int k = 0; k < 8; ++k) s_q[i + k] = v[k];
         }
     }
-    for (uint32_t i = tid; i < group * D; i += RW_THREADS) s_o[i] = 0.0f;
-    for (uint32_t i = tid; i < group; i += RW_THREADS) { s_m[i] = -INFINITY; s_l[i] = 0.0f; }
     __syncthreads();
     for (uint32_t j0 = j_lo; j0 < j_hi; j0 += RW_SC) {
         const uint32_t n = min(RW_SC, j_hi - j0);
         // scores: four lanes per key, sixteen keys per warp and step
         const uint32_t sub = lane & 3u, ki = lane >> 2;
+#pragma unroll 1
         for (uint32_t b = warp * 16; b < n; b += RW_THREADS / 2) {
             const uint32_t ja = b + ki, jb = b + 8 + ki;
             const T *ka = kc + (size_t)a.ring.slot_of_pos(j0 + min(ja, n - 1)) * D, *kb = kc + (size_t)a.ring.slot_of_pos(j0 + min(jb, n - 1)) * D;
-            for (uint32_t h0 = 0; h0 < group; h0 += RW_HB) {
-                float da[RW_HB], db[RW_HB];
+#pragma unroll 1
+            for (uint32_t h0 = 0; h0 < group; h0 += HB) {
+                float da[HB], db[HB];
 #pragma unroll
-                for (uint32_t h = 0; h < RW_HB; ++h) da[h] = db[h] = 0.0f;
+                for (uint32_t h = 0; h < HB; ++h) da[h] = db[h] = 0.0f;
 #pragma unroll
                 for (uint32_t c = 0; c < D / 32; ++c) {
                     float va[8], vb[8];
@@ -133,8 +152,7 @@ __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams
                     get8(ka + k, va);
                     get8(kb + k, vb);
 #pragma unroll
-                    for (uint32_t h = 0; h < RW_HB; ++h) {
-                        if (h0 + h >= group) break;
+                    for (uint32_t h = 0; h < HB; ++h) {
                         const float4 q0 = *reinterpret_cast<const float4 *>(s_q + (h0 + h) * D + k), q1 = *reinterpret_cast<const float4 *>(s_q + (h0 + h) * D + k + 4);
                         const float q[8] = {q0.x, q0.y, q0.z, q0.w, q1.x, q1.y, q1.z, q1.w};
 #pragma unroll
@@ -142,21 +160,24 @@ __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams
                     }
                 }
 #pragma unroll
-                for (uint32_t h = 0; h < RW_HB; ++h) {
-                    if (h0 + h >= group) break;
-                    float u = da[h], w = db[h];
-                    u = __fadd_rn(u, __shfl_xor_sync(0xffffffffu, u, 1)); w = __fadd_rn(w, __shfl_xor_sync(0xffffffffu, w, 1));
-                    u = __fadd_rn(u, __shfl_xor_sync(0xffffffffu, u, 2)); w = __fadd_rn(w, __shfl_xor_sync(0xffffffffu, w, 2));
-                    if (sub == (h & 3u)) {
-                        const uint32_t hh = g * group + h0 + h;
-                        const float sc = __ldg(a.head_scale + hh), sl = __ldg(a.head_slope + hh);
-                        if (ja < n) s_p[(h0 + h) * RW_SC + ja] = u * sc - sl * (float)(pos - (j0 + ja));
-                        if (jb < n) s_p[(h0 + h) * RW_SC + jb] = w * sc - sl * (float)(pos - (j0 + jb));
+                for (int m = 1; m < 4; m <<= 1)
+#pragma unroll
+                    for (uint32_t h = 0; h < HB; ++h) {
+                        da[h] = __fadd_rn(da[h], __shfl_xor_sync(0xffffffffu, da[h], m));
+                        db[h] = __fadd_rn(db[h], __shfl_xor_sync(0xffffffffu, db[h], m));
                     }
-                }
+#pragma unroll
+                for (uint32_t h = 0; h < HB; ++h)
+                    if (sub == (h & 3u)) {
+                        const uint32_t hh = g * group + min(h0 + h, group - 1);
+                        const float sc = __ldg(a.head_scale + hh), sl = __ldg(a.head_slope + hh);
+                        if (ja < n) s_p[(h0 + h) * RW_SC + ja] = da[h] * sc - sl * (float)(pos - (j0 + ja));
+                        if (jb < n) s_p[(h0 + h) * RW_SC + jb] = db[h] * sc - sl * (float)(pos - (j0 + jb));
+                    }
             }
         }
         __syncthreads();
+#pragma unroll 1
         for (uint32_t h = warp; h < group; h += RW_THREADS / 32) {          // softmax terms of the tile, one warp per head
             float mx = -INFINITY;
             for (uint32_t j = lane; j < n; j += 32) mx = fmaxf(mx, s_p[h * RW_SC + j]);
@@ -169,66 +190,68 @@ __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams
             if (lane == 0) { const float al = expf(m_old - m_new); s_al[h] = al; s_m[h] = m_new; s_l[h] = s_l[h] * al + sum; }
         }
         __syncthreads();
-        // values: thread = (key slice, eight columns)
+        // values: thread = (key slice, eight columns); padding heads multiply finite leftovers that nobody reads
         constexpr uint32_t CPK = D / 8, KS = RW_THREADS / CPK;
         const uint32_t ks = tid / CPK, c = tid % CPK;
-        for (uint32_t h0 = 0; h0 < group; h0 += RW_PB) {
-            float acc[RW_PB][8];
+#pragma unroll 1
+        for (uint32_t h0 = 0; h0 < group; h0 += HB) {
+            float acc[HB][8];
 #pragma unroll
-            for (uint32_t h = 0; h < RW_PB; ++h)
+            for (uint32_t h = 0; h < HB; ++h)
 #pragma unroll
                 for (int i = 0; i < 8; ++i) acc[h][i] = 0.0f;
-            if (ks < KS)
+            if (ks < KS) {
 #pragma unroll 4
                 for (uint32_t j = ks; j < n; j += KS) {
                     float v[8];
                     get8(vc + (size_t)a.ring.slot_of_pos(j0 + j) * D + c * 8, v);
 #pragma unroll
-                    for (uint32_t h = 0; h < RW_PB; ++h) {
-                        if (h0 + h >= group) break;
+                    for (uint32_t h = 0; h < HB; ++h) {
                         const float e = s_p[(h0 + h) * RW_SC + j];
 #pragma unroll
                         for (int i = 0; i < 8; ++i) acc[h][i] = __fmaf_rn(e, v[i], acc[h][i]);
                     }
                 }
 #pragma unroll
-            for (uint32_t h = 0; h < RW_PB; ++h) {
-                if (h0 + h >= group) break;
-                if (ks < KS)
-#pragma unroll
-                    for (int i = 0; i < 8; ++i) s_red[ks * D + c * 8 + i] = acc[h][i];
-                __syncthreads();
-                for (uint32_t d = tid; d < D; d += RW_THREADS) {
-                    float o = 0.0f;
-                    for (uint32_t k = 0; k < KS; ++k) o = __fadd_rn(o, s_red[k * D + d]);
-                    s_o[(h0 + h) * D + d] = s_o[(h0 + h) * D + d] * s_al[h0 + h] + o;
+                for (uint32_t h = 0; h < HB; ++h) {
+                    float4 *dst = reinterpret_cast<float4 *>(s_red + (ks * HB + h) * D + c * 8);
+                    dst[0] = make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]);
+                    dst[1] = make_float4(acc[h][4], acc[h][5], acc[h][6], acc[h][7]);
                 }
-                __syncthreads();
             }
+            __syncthreads();
+            for (uint32_t e = tid; e < HB * D; e += RW_THREADS) {
+                float o = 0.0f;
+#pragma unroll 8
+                for (uint32_t k = 0; k < KS; ++k) o = __fadd_rn(o, s_red[k * HB * D + e]);
+                s_o[h0 * D + e] = s_o[h0 * D + e] * s_al[h0 + e / D] + o;
+            }
+            __syncthreads();
         }
     }
-    // merge over the cluster: CTA r finishes the group's heads r, r + cs, ..
+    // merge over the cluster: factors of every (head, CTA), then the outputs shared out over all CTAs
+    __syncthreads();
     if (cs > 1) cluster_sync_all();
-    for (uint32_t h = me; h < group; h += cs) {
+    for (uint32_t i = tid; i < group * cs; i += RW_THREADS) {
+        const uint32_t h = i / cs, r = i % cs;
+        s_fm[h * RW_MAX_CS + r] = cs > 1 ? ld_cluster_f32(s_m + h, r) : s_m[h];
+        s_fl[h * RW_MAX_CS + r] = cs > 1 ? ld_cluster_f32(s_l + h, r) : s_l[h];
+    }
+    __syncthreads();
+    for (uint32_t h = tid; h < group; h += RW_THREADS) {
         float m = -INFINITY, l = 0.0f;
-        for (uint32_t r = 0; r < cs; ++r) m = fmaxf(m, cs > 1 ? ld_cluster_f32(s_m + h, r) : s_m[h]);
-        float f[16];
+        for (uint32_t r = 0; r < cs; ++r) m = fmaxf(m, s_fm[h * RW_MAX_CS + r]);
+        for (uint32_t r = 0; r < cs; ++r) { const float f = expf(s_fm[h * RW_MAX_CS + r] - m); s_fm[h * RW_MAX_CS + r] = f; l += f * s_fl[h * RW_MAX_CS + r]; }
+        s_fl[h * RW_MAX_CS] = 1.0f / l;
+    }
+    __syncthreads();
+    for (uint32_t e = me * RW_THREADS + tid; e < group * a.vdim; e += cs * RW_THREADS) {
+        const uint32_t h = e / a.vdim, d = e % a.vdim;
+        float o = 0.0f;
 #pragma unroll
-        for (uint32_t r = 0; r < 16; ++r) {
-            f[r] = 0.0f;
-            if (r < cs) {
-                f[r] = expf((cs > 1 ? ld_cluster_f32(s_m + h, r) : s_m[h]) - m);
-                l += f[r] * (cs > 1 ? ld_cluster_f32(s_l + h, r) : s_l[h]);
-            }
-        }
-        const float inv = 1.0f / l;
-        for (uint32_t d = tid; d < a.vdim; d += RW_THREADS) {
-            float o = 0.0f;
-#pragma unroll
-            for (uint32_t r = 0; r < 16; ++r)
-                if (r < cs) o = __fmaf_rn(f[r], cs > 1 ? ld_cluster_f32(s_o + h * D + d, r) : s_o[h * D + d], o);
-            act_store<sizeof(T) == 4>(a.out, t, (g * group + h) * a.vdim + d, o * inv);
-        }
+        for (uint32_t r = 0; r < RW_MAX_CS; ++r)
+            if (r < cs) o = __fmaf_rn(s_fm[h * RW_MAX_CS + r], cs > 1 ? ld_cluster_f32(s_o + h * D + d, r) : s_o[h * D + d], o);
+        act_store<sizeof(T) == 4>(a.out, t, (g * group + h) * a.vdim + d, o * s_fl[h * RW_MAX_CS]);
     }
     if (cs > 1) cluster_sync_all();
 }
@@ -249,6 +272,8 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
+
+__device__ __forceinline__ float fl_exp2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
 template <int D>
 __global__ void __launch_bounds__(FL_THREADS) window_flash_kernel(const AttnParams p) {
@@ -288,7 +313,7 @@ __global__ void __launch_bounds__(FL_THREADS) window_flash_kernel(const AttnPara
         sc[i] = __ldg(a.head_scale + g * group + r % group) * LOG2E;
         sl[i] = __ldg(a.head_slope + g * group + r % group) * LOG2E;
     }
-    const uint32_t window = a.ring.window ? a.ring.window : 0xffffffffu;
+    const uint32_t window = a.ring.window ? a.ring.window : 0x7fffffffu;
     // positions some row of this warp can see
     const uint32_t w_first = pos0 + min(r0 + warp * 16, rows - 1) / group, w_last = pos0 + min(r0 + warp * 16 + 15, rows - 1) / group;
     const uint32_t w_lo = w_first + 1 - a.ring.active_len(w_first + 1);
@@ -319,33 +344,44 @@ __global__ void __launch_bounds__(FL_THREADS) window_flash_kernel(const AttnPara
             }
         }
         float mx[2] = {-INFINITY, -INFINITY};
+        // bias of the tile's first key of this thread, the others follow in exact steps (small integers times the slope)
+        const float f0[2] = {(float)(int)(j0 + (lane & 3u) * 2 - qpos[0]), (float)(int)(j0 + (lane & 3u) * 2 - qpos[1])};
 #pragma unroll
         for (uint32_t n = 0; n < FL_N / 8; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const uint32_t i = e >> 1, j = j0 + n * 8 + (lane & 3u) * 2 + (e & 1);
-                const uint32_t dist = qpos[i] - j;            // wraps for later positions: larger than any window
-                const bool seen = j <= qpos[i] && dist < window;
-                const float v = seen ? __fmaf_rn(s[n][e], sc[i], -sl[i] * (float)dist) : -INFINITY;
-                s[n][e] = v;
-                mx[i] = fmaxf(mx[i], v);
+                const uint32_t i = e >> 1;
+                s[n][e] = __fmaf_rn(s[n][e], sc[i], sl[i] * (f0[i] + (float)(n * 8 + (e & 1))));
             }
+        if (j0 + FL_N - 1 > w_first || w_last >= j0 + window) {            // some key of the tile is out of some row's sight
+#pragma unroll
+            for (uint32_t n = 0; n < FL_N / 8; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const uint32_t i = e >> 1, j = j0 + n * 8 + (lane & 3u) * 2 + (e & 1);
+                    if (j > qpos[i] || qpos[i] - j >= window) s[n][e] = -INFINITY;
+                }
+        }
+#pragma unroll
+        for (uint32_t n = 0; n < FL_N / 8; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
         float al[2];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
             mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
             const float m_new = fmaxf(m[i], mx[i]);
-            al[i] = m_new == -INFINITY ? 1.0f : exp2f(m[i] - m_new);
+            al[i] = m_new == -INFINITY ? 1.0f : fl_exp2(m[i] - m_new);
             m[i] = m_new;
             l[i] *= al[i];
         }
+        const float mm[2] = {m[0] == -INFINITY ? 0.0f : m[0], m[1] == -INFINITY ? 0.0f : m[1]};        // a row that has seen nothing yet: exp2(-inf) = 0
 #pragma unroll
         for (uint32_t n = 0; n < FL_N / 8; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const float mm = m[e >> 1];
-                const float v = mm == -INFINITY ? 0.0f : exp2f(s[n][e] - mm);
+                const float v = fl_exp2(s[n][e] - mm[e >> 1]);
                 s[n][e] = v;
                 l[e >> 1] += v;
             }
@@ -385,17 +421,26 @@ __global__ void __launch_bounds__(FL_THREADS) window_flash_kernel(const AttnPara
     }
 }
 
-template <typename T, int D>
-cudaError_t row_launch(cudaStream_t s, const AttnParams &p, int sm_count, bool pdl) {
+template <typename T, int D, int HB>
+cudaError_t row_launch_hb(cudaStream_t s, const AttnParams &p, int sm_count, bool pdl) {
     const WindowAttnArgs &a = p.a;
-    const uint32_t group = a.n_q / a.n_kv;
     uint32_t cs = 1;                            // CTAs per (token, kv head): at least 64 positions each, about one wave of CTAs
     const uint32_t longest = a.ring.window ? a.ring.window : p.ring_rows;
-    while (cs < 8 && cs * 2 * 64 <= longest && cs * 2 * a.n_kv * p.n_tok <= (uint32_t)sm_count) cs *= 2;
-    const size_t smem = rw_smem(group, D);
-    cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(window_row_kernel<T, D>), smem);
+    while (cs < RW_MAX_CS && cs * 2 * 64 <= longest && cs * 2 * a.n_kv * p.n_tok <= (uint32_t)sm_count) cs *= 2;
+    const size_t smem = rw_smem(a.n_q / a.n_kv, D, HB);
+    cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(window_row_kernel<T, D, HB>), smem);
     if (e != cudaSuccess) return e;
-    return launch_cluster(window_row_kernel<T, D>, dim3(cs, a.n_kv, p.n_tok), dim3(RW_THREADS), smem, s, pdl, cs, p);
+    return launch_cluster(window_row_kernel<T, D, HB>, dim3(cs, a.n_kv, p.n_tok), dim3(RW_THREADS), smem, s, pdl, cs, p);
+}
+inline uint32_t head_pass(bool f32, uint32_t group) { return f32 ? 4u : group == 1 ? 1u : group <= 4 ? 4u : 8u; }
+template <int D>
+cudaError_t row_launch(cudaStream_t s, bool f32, const AttnParams &p, int sm_count, bool pdl) {
+    if (f32) return row_launch_hb<float, D, 4>(s, p, sm_count, pdl);
+    switch (head_pass(false, p.a.n_q / p.a.n_kv)) {
+        case 1: return row_launch_hb<__nv_bfloat16, D, 1>(s, p, sm_count, pdl);
+        case 4: return row_launch_hb<__nv_bfloat16, D, 4>(s, p, sm_count, pdl);
+        default: return row_launch_hb<__nv_bfloat16, D, 8>(s, p, sm_count, pdl);
+    }
 }
 template <int D>
 cudaError_t flash_launch(cudaStream_t s, const AttnParams &p, bool pdl) {
@@ -414,17 +459,19 @@ uint32_t window_attn_row(uint32_t dim, uint32_t vdim) {
     return 0;
 }
 
+bool window_attn_fits(bool f32, uint32_t group, uint32_t row) { return rw_smem(group, row, head_pass(f32, group)) <= 224 * 1024; }
+
 cudaError_t launch_window_attention(cudaStream_t s, bool f32, const WindowAttnArgs &a, uint32_t n_tok, int sm_count, uint32_t *launches, bool pdl) {
     AttnParams p{a, n_tok, 0, n_tok == 1 ? 1u : 0u};
     p.ring_rows = a.ring.ring_len;
-    if (n_tok > 65535u || rw_smem(a.n_q / a.n_kv, a.row) > 220 * 1024) return cudaErrorInvalidValue;
+    if (n_tok > 65535u || !window_attn_fits(f32, a.n_q / a.n_kv, a.row)) return cudaErrorInvalidValue;
     *launches = n_tok == 1 ? 1 : 2;
     if (n_tok > 1) {
         const dim3 grid((a.n_q + 2 * a.n_kv + 7) / 8, n_tok);
         cudaError_t e = f32 ? launch_kernel(window_prep_kernel<float>, grid, dim3(256), 0, s, pdl, p) : launch_kernel(window_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl, p);
         if (e != cudaSuccess) return e;
     }
-#define K2T_ROW(D) case D: return f32 ? row_launch<float, D>(s, p, sm_count, pdl) : n_tok == 1 ? row_launch<__nv_bfloat16, D>(s, p, sm_count, pdl) : flash_launch<D>(s, p, pdl)
+#define K2T_ROW(D) case D: return f32 || n_tok == 1 ? row_launch<D>(s, f32, p, sm_count, pdl) : flash_launch<D>(s, p, pdl)
     switch (a.row) {
         K2T_ROW(32);
         K2T_ROW(64);

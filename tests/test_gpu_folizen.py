@@ -199,8 +199,8 @@ def test_state_far_back(engine):
     t = model["tensors"]
     t["l0.mix.w0"][:] = -12.0
     t["l0.mix.a.b"][:] = -9.0
-    t["l0.mix.v"][:] *= fm.bf16(np.float32(0.02))
-    t["embed"][1] *= fm.bf16(np.float32(50))
+    t["l0.mix.v"][:] = fm.bf16(0.02 * t["l0.mix.v"])
+    t["embed"][1] = fm.bf16(50 * t["embed"][1])
     toks = tokens_of(model, 1200, seed=6) % 28 + 2
     plain, _ = ref.forward(model, toks)
     toks[3] = 1
