@@ -66,8 +66,10 @@ __global__ void __launch_bounds__(1024) block_norm_kernel(float *__restrict__ x,
     }
 }
 
-// A cluster of `cs` CTAs per token; CTA r holds the panels [r np / cs, (r + 1) np / cs) of the vector.  Three exchanges over
-// distributed shared memory: the sublayer's sum of squares, the partial gate products, the token input's sum of squares.
+// A cluster of `cs` CTAs per token; CTA r holds the panels [r np / cs, (r + 1) np / cs) of the vector.  Two exchanges over
+// distributed shared memory: the sublayer's sum of squares together with the partial gate products - of x and of y w apart, so
+// that the products need not wait for the norm: gate (x + y w / rms) = gate x + gate (y w) / rms - and the token input's sum of
+// squares.
 // The CTA's share of both weight matrices is bulk-copied to shared memory before the dependency wait (STAGED: bf16 panels that
 // fit), so after the wait only the two vectors come from global memory.
 constexpr uint32_t NS_THREADS = 256;
@@ -77,7 +79,7 @@ constexpr uint32_t NS_WAIT_LIMIT = 1u << 22;
 __host__ __device__ inline uint32_t ns_slice_panels(uint32_t np, uint32_t cs) { return (np + cs - 1) / cs; }
 inline size_t ns_vec_smem(uint32_t n, uint32_t dim, uint32_t cs) {
     const uint32_t slice = ns_slice_panels((n + 63) / 64, cs) * 64, dp = (dim + 63) / 64 * 64;
-    return (((size_t)2 * slice + dp + (size_t)cs * dim) * 4 + 127) & ~(size_t)127;
+    return (((size_t)2 * slice + dp + (size_t)2 * cs * dim) * 4 + 127) & ~(size_t)127;
 }
 inline size_t ns_weight_smem(uint32_t n, uint32_t dim, uint32_t cs) {
     const uint32_t sp = ns_slice_panels((n + 63) / 64, cs), dp = (dim + 63) / 64;
@@ -93,7 +95,7 @@ __global__ void __launch_bounds__(NS_THREADS) norm_side_kernel(float *__restrict
     const uint32_t cs = cluster_size(), me = cluster_rank(), t = blockIdx.x / cs, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const uint32_t np = (n + 63) / 64, sp = ns_slice_panels(np, cs), p0 = min(np, me * sp), p1 = min(np, p0 + sp);
     const uint32_t slice = sp * 64, dim = sd.dim, dp = (dim + 63) / 64 * 64;
-    float *s_x = sm, *s_y = s_x + slice, *s_g = s_y + slice, *s_part = s_g + dp;      // s_part [cs][dim]: written by the peers
+    float *s_x = sm, *s_y = s_x + slice, *s_g = s_y + slice, *s_part = s_g + dp;      // s_part [cs][2 dim]: written by the peers
     const uint32_t k0 = p0 * 64, k1 = min(n, p1 * 64);
     DenseView gate = sd.gate, proj = sd.proj;
     const uint32_t bar = (uint32_t)__cvta_generic_to_shared(&bar_w);
@@ -112,52 +114,66 @@ __global__ void __launch_bounds__(NS_THREADS) norm_side_kernel(float *__restrict
         gate.base = s_w; gate.rows_pad = dim;
         proj.base = s_w + mine * dim * 128; proj.rows_pad = mine * 64;
     }
-    for (uint32_t i = tid; i < slice; i += NS_THREADS) s_x[i] = 0.0f;
+    for (uint32_t i = tid; i < 2 * slice; i += NS_THREADS) s_x[i] = 0.0f;      // s_x and s_y
     for (uint32_t i = tid; i < dp; i += NS_THREADS) s_g[i] = 0.0f;
+    float w_first = 0.0f, n_first = 0.0f;       // the norm weights of the thread's first element
+    if (k0 + tid < k1) { w_first = __ldg(w + k0 + tid); n_first = __ldg(sd.norm + k0 + tid); }
+    if (cs > 1) cluster_sync_all();             // every CTA of the cluster runs before its shared memory is written from outside
     pdl_wait();
     pdl_trigger();
-    if (cs > 1) cluster_sync_all();             // every CTA of the cluster runs before its shared memory is written from outside
     float *xr = x + t * x_stride;
     const float *yr = y + t * y_stride;
     const uint16_t *e = sd.table + (size_t)__ldcg(sd.tokens + t) * sd.table_stride + sd.offset;
     const float e_first = tid < dim ? bf16_bits_to_f32(__ldg(e + tid)) : 0.0f;
-    // sublayer output: x + y / rms(y) * w
     float ss[1] = {0.0f};
     for (uint32_t k = k0 + tid; k < k1; k += NS_THREADS) {
         const float v = __ldcg(yr + k);
         s_x[k - k0] = __ldcg(xr + k);
-        s_y[k - k0] = v;
+        s_y[k - k0] = v * (k == k0 + tid ? w_first : __ldg(w + k));
         ss[0] = __fmaf_rn(v, v, ss[0]);
     }
-    block_sum<1>(ss, scratch);
-    cluster_sum<1>(ss, slot_a);
-    const float inv = 1.0f / sqrtf(ss[0] / (float)n + eps);
-    for (uint32_t k = k0 + tid; k < k1; k += NS_THREADS) s_x[k - k0] += s_y[k - k0] * inv * __ldg(w + k);
     if (STAGED) {
         bool ok = false;
         for (uint32_t spin = 0; spin < NS_WAIT_LIMIT && !ok; ++spin) ok = mbar_try_wait(bar, 0u);
         if (!ok && err_flag != nullptr) atomicExch(err_flag, 1u);
     }
-    __syncthreads();
+    block_sum<1>(ss, scratch);                  // its barriers also publish s_x and s_y
     // partial gate products of the slice: eight lanes per row, four rows per warp and step
     const uint32_t sub = lane & 7u, q0 = STAGED ? 0u : p0, q1 = STAGED ? p1 - p0 : p1;
-#pragma unroll 2
+    // (loops kept rolled: the kernel runs its code once per launch, and instruction fetch is what unrolled copies cost)
+#pragma unroll 1
     for (uint32_t r0 = warp * 4; r0 < dim; r0 += NS_THREADS / 8) {
-        const uint32_t r = r0 + (lane >> 3);
-        const float d = row_dot8<F32, STAGED>(gate, min(r, dim - 1), q0, q1, s_x, sub);
-        if (r < dim && sub < cs) st_cluster_f32(s_part + (size_t)me * dim + r, sub, d);
+        const uint32_t r = r0 + (lane >> 3), rr = min(r, dim - 1);
+        float dx = 0.0f, dy = 0.0f;
+        if (STAGED) {
+            const uint4 *q = static_cast<const uint4 *>(gate.base) + (size_t)rr * 8 + (sub ^ (rr & 7u));
+#pragma unroll 1
+            for (uint32_t k = sub * 8; k < (p1 - p0) * PANEL; k += PANEL, q += (size_t)dim * 8) {
+                const uint4 v = *q;
+                dx = dot8(v, s_x + k, dx);
+                dy = dot8(v, s_y + k, dy);
+            }
+#pragma unroll
+            for (int m = 1; m < 8; m <<= 1) { dx = __fadd_rn(dx, __shfl_xor_sync(0xffffffffu, dx, m)); dy = __fadd_rn(dy, __shfl_xor_sync(0xffffffffu, dy, m)); }
+        } else {
+            dx = row_dot8<F32>(gate, rr, q0, q1, s_x, sub);
+            dy = row_dot8<F32>(gate, rr, q0, q1, s_y, sub);
+        }
+        if (r < dim && sub < cs) { st_cluster_f32(s_part + ((size_t)me * 2) * dim + r, sub, dx); st_cluster_f32(s_part + ((size_t)me * 2 + 1) * dim + r, sub, dy); }
     }
-    if (cs > 1) cluster_sync_all();
-    else __syncthreads();
+    if (cs == 1) __syncthreads();
+    cluster_sum<1>(ss, slot_a);                 // its barrier also publishes the partial products
+    const float inv = rsqrtf(ss[0] / (float)n + eps);
     for (uint32_t i = tid; i < dim; i += NS_THREADS) {
-        float z = 0.0f;
-        for (uint32_t r = 0; r < cs; ++r) z = __fadd_rn(z, s_part[(size_t)r * dim + i]);
-        s_g[i] = gelu_tanh(z) * (i == tid ? e_first : bf16_bits_to_f32(__ldg(e + i)));
+        float zx = 0.0f, zy = 0.0f;
+        for (uint32_t r = 0; r < cs; ++r) { zx = __fadd_rn(zx, s_part[((size_t)r * 2) * dim + i]); zy = __fadd_rn(zy, s_part[((size_t)r * 2 + 1) * dim + i]); }
+        s_g[i] = gelu_tanh(__fmaf_rn(zy, inv, zx)) * (i == tid ? e_first : bf16_bits_to_f32(__ldg(e + i)));
     }
+    for (uint32_t k = tid; k < k1 - k0 && k1 > k0; k += NS_THREADS) s_x[k] = __fmaf_rn(s_y[k], inv, s_x[k]);
     __syncthreads();
     float s2[1] = {0.0f};
     const uint32_t row_off = STAGED ? k0 : 0u;
-#pragma unroll 4
+#pragma unroll 1
     for (uint32_t r0 = k0 + warp * 4; r0 < k1; r0 += NS_THREADS / 8) {
         const uint32_t r = r0 + (lane >> 3);
         const float d = row_dot8<F32, STAGED>(proj, min(r, k1 - 1) - row_off, 0, proj.panels, s_g, sub);
@@ -165,9 +181,9 @@ __global__ void __launch_bounds__(NS_THREADS) norm_side_kernel(float *__restrict
     }
     block_sum<1>(s2, scratch);
     cluster_sum<1>(s2, slot_b);
-    const float inv2 = 1.0f / sqrtf(s2[0] / (float)n + eps);
+    const float inv2 = rsqrtf(s2[0] / (float)n + eps);
     for (uint32_t k = k0 + tid; k < k1; k += NS_THREADS) {
-        const float v = s_x[k - k0] + s_y[k - k0] * inv2 * __ldg(sd.norm + k);
+        const float v = s_x[k - k0] + s_y[k - k0] * inv2 * (k == k0 + tid ? n_first : __ldg(sd.norm + k));
         xr[k] = v;
         act_store<F32>(out, t, k, v);
     }
@@ -192,9 +208,9 @@ __global__ void __launch_bounds__(256) polynorm_kernel(const float *__restrict__
     const uint32_t np = (n + 63) / 64, p0 = min(np, me * ns_slice_panels(np, cs)), p1 = min(np, p0 + ns_slice_panels(np, cs));
     const uint32_t k0 = p0 * 64 + threadIdx.x * 4, k1 = min(n, p1 * 64);
     const float ca = __ldg(coef), cb = __ldg(coef + 1), cc = __ldg(coef + 2), ce = __ldg(coef + 3);
+    if (cs > 1) cluster_sync_all();
     pdl_wait();
     pdl_trigger();
-    if (cs > 1) cluster_sync_all();
     const float *zr = z + t * z_stride;
     float m[3] = {0.0f, 0.0f, 0.0f};             // sums of z^2, z^4, z^6
     constexpr uint32_t KEEP = 8;

@@ -44,6 +44,7 @@ struct WindowAttnArgs {
     KvRing ring;                       // sinks 0; window 0 = every earlier position
     float eps;
     Act out;                           // [n_tok][n_q * vdim]
+    uint32_t *err_flag;
 };
 bool window_attn_fits(bool f32, uint32_t group, uint32_t row);       // queries of a group beside one another in shared memory
 uint32_t window_attn_row(uint32_t dim, uint32_t vdim);       // cache row in elements; 0 = larger than the kernels support
@@ -70,6 +71,6 @@ size_t delta_record_floats(uint32_t n_tok, uint32_t heads, uint32_t drow);
 bool delta_step_fits(const DeltaArgs &a);
 cudaError_t launch_delta_step(cudaStream_t s, bool f32, const DeltaArgs &a, bool pdl);                                   // one token, one launch
 cudaError_t launch_delta_tanh(cudaStream_t s, bool f32, const DeltaArgs &a, const Act &out, uint32_t n_tok, bool pdl);   // activation of the decay product
-cudaError_t launch_delta_prompt(cudaStream_t s, bool f32, const DeltaArgs &a, uint32_t n_tok, bool pdl);                 // three launches
+cudaError_t launch_delta_prompt(cudaStream_t s, bool f32, const DeltaArgs &a, uint32_t n_tok, int sm_count, bool pdl);   // three launches
 
 }  // namespace k2t

@@ -73,7 +73,7 @@ bool mix_attention(KronosCudaEngine *e, Block &B, uint32_t T, const Act &out) {
     a.qkv = b.z; a.qkv_stride = b.zs;
     a.q_norm = B.q_norm; a.k_norm = B.k_norm; a.head_scale = B.head_scale; a.head_slope = B.head_slope;
     a.k_cache = B.k; a.v_cache = B.v; a.q = b.q; a.pos = e->d_pos;
-    a.n_q = B.heads; a.n_kv = B.kv_heads; a.dim = B.dim; a.vdim = B.vdim; a.row = B.row; a.ring = B.ring; a.eps = e->cfg.rms_norm_eps; a.out = out;
+    a.n_q = B.heads; a.n_kv = B.kv_heads; a.dim = B.dim; a.vdim = B.vdim; a.row = B.row; a.ring = B.ring; a.eps = e->cfg.rms_norm_eps; a.out = out; a.err_flag = e->ctx->d_err;
     uint32_t n = 0;
     const cudaError_t err = launch_window_attention(e->ctx->stream, b.f32, a, T, e->ctx->sm_count, &n, e->pdl);
     return engine_count(e, err, "attention", n);
@@ -91,7 +91,7 @@ bool mix_delta(KronosCudaEngine *e, Block &B, uint32_t T, const Act &out) {
     if (T == 1 && delta_step_fits(a)) return engine_count(e, launch_delta_step(s, b.f32, a, e->pdl), "recurrence");
     const Act r = act_of(b, b.act_s, T, B.rank);
     return engine_count(e, launch_delta_tanh(s, b.f32, a, r, T, e->pdl), "decay tanh") && product(e, B.decay, r, T, b.logit, b.ls, "decay product") &&
-           engine_count(e, launch_delta_prompt(s, b.f32, a, T, e->pdl), "recurrence", 3);
+           engine_count(e, launch_delta_prompt(s, b.f32, a, T, e->ctx->sm_count, e->pdl), "recurrence", 3);
 }
 
 bool norm_add(KronosCudaEngine *e, const float *w, const Act &out, uint32_t T) {

@@ -50,7 +50,7 @@ template <bool F32, bool SHARED = false> __device__ __forceinline__ float row_do
         for (uint32_t k = p0 * PANEL + sub; k < k1; k += 8) acc = __fmaf_rn(__ldg(w + k), x[k - p0 * PANEL], acc);
     } else {
         const uint4 *w = static_cast<const uint4 *>(m.base);
-#pragma unroll 4
+#pragma unroll SHARED ? 1 : 4
         for (uint32_t p = p0; p < p1; ++p) {
             const uint4 *q = w + ((size_t)p * m.rows_pad + row) * 8 + (sub ^ (row & 7u));
             acc = dot8(SHARED ? *q : __ldg(q), x + (p - p0) * PANEL + sub * 8, acc);

@@ -1325,7 +1325,7 @@ int32_t kronos_cuda_engine_decode_greedy(KronosCudaEngine *e, uint32_t first_tok
         std::vector<unsigned long long> h(tl_cap + 2);
         cudaMemcpy(h.data(), tl_dev, h.size() * 8, cudaMemcpyDeviceToHost);
         cudaFree(tl_dev);
-        const int which = (pos_start + 1 > ATTN_EXACT_CTX || e->ring.window) ? 1 : 0;
+        const int which = !e->blocks && (pos_start + 1 > ATTN_EXACT_CTX || e->ring.window) ? 1 : 0;
         const std::vector<const char *> &lab = e->tl_labels[which];
         const size_t n = std::min<size_t>(h[0], tl_cap);
         std::sort(h.begin() + 2, h.begin() + 2 + n);

@@ -80,47 +80,65 @@ __global__ void __launch_bounds__(256) window_prep_kernel(const AttnParams p) {
 
 // ------------------------------------------------------------------------------------------------ one token per cluster
 // The heads of a group run in passes of HB (the group is padded to full passes with zero queries), so the inner loops carry no
-// branches and a step's row loads are all in flight together.  A decode step pulls the cached rows it will read towards L2 before
-// its dependency wait: they were written by earlier steps, only the new row depends on the predecessor.
-constexpr uint32_t RW_THREADS = 256, RW_SC = 256, RW_MAX_CS = 8;
+// branches.  Cached rows come in tiles by bulk copy (a CTA's positions are consecutive, so a tile is one run of the ring, two
+// where it wraps); a decode step asks for its first tiles before its dependency wait - earlier steps wrote those rows - and lays
+// the new position's row over the stale one once the tile has landed.
+constexpr uint32_t RW_THREADS = 256, RW_MAX_CS = 8;
+constexpr uint32_t RW_WAIT_LIMIT = 1u << 22;
+// positions per tile: 64 KiB of keys (32 for long passes and fp32 rows), at most 256, a multiple of 16
+template <typename T> __host__ __device__ constexpr uint32_t rw_tile(uint32_t row, uint32_t hb) {
+    const uint32_t n = (hb > 4 || sizeof(T) == 4 ? 32768u : 65536u) / (row * (uint32_t)sizeof(T));
+    return (n > 256u ? 256u : n) & ~15u;
+}
 __host__ __device__ inline uint32_t rw_pad(uint32_t group, uint32_t hb) { return (group + hb - 1) / hb * hb; }
-inline size_t rw_smem(uint32_t group, uint32_t row, uint32_t hb) {
-    return ((size_t)rw_pad(group, hb) * (2 * row + RW_SC + 4 + 2 * RW_MAX_CS) + (size_t)8 * RW_THREADS * hb) * 4;
+template <typename T> inline size_t rw_smem(uint32_t group, uint32_t row, uint32_t hb) {
+    const uint32_t tile = rw_tile<T>(row, hb);
+    return (size_t)2 * tile * row * sizeof(T) + ((size_t)rw_pad(group, hb) * (2 * row + tile + 4 + 2 * RW_MAX_CS) + (size_t)8 * RW_THREADS * hb + 2 * row) * 4;
 }
 
 template <typename T, int D, int HB>
 __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams p) {
-    extern __shared__ __align__(16) float sm[];
+    extern __shared__ __align__(128) uint8_t smb[];
+    __shared__ __align__(8) uint64_t bars[2];
+    constexpr uint32_t TILE = rw_tile<T>(D, HB);
     const WindowAttnArgs &a = p.a;
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, cs = cluster_size(), me = cluster_rank();
     const uint32_t g = blockIdx.y, t = blockIdx.z, group = a.n_q / a.n_kv, gp = rw_pad(group, HB);
-    float *s_q = sm, *s_o = s_q + gp * D, *s_p = s_o + gp * D, *s_red = s_p + gp * RW_SC, *s_m = s_red + 8 * RW_THREADS * HB, *s_l = s_m + gp, *s_al = s_l + gp,
-          *s_fm = s_al + 2 * gp, *s_fl = s_fm + gp * RW_MAX_CS;
+    T *s_k = reinterpret_cast<T *>(smb), *s_v = s_k + TILE * D;
+    float *s_q = reinterpret_cast<float *>(s_v + TILE * D), *s_o = s_q + gp * D, *s_red = s_o + gp * D, *s_new = s_red + 8 * RW_THREADS * HB, *s_p = s_new + 2 * D, *s_m = s_p + gp * TILE,
+          *s_l = s_m + gp, *s_al = s_l + gp, *s_fm = s_al + 2 * gp, *s_fl = s_fm + gp * RW_MAX_CS;
     T *kc = static_cast<T *>(a.k_cache) + (size_t)g * p.ring_rows * D, *vc = static_cast<T *>(a.v_cache) + (size_t)g * p.ring_rows * D;
+    const uint32_t bar = (uint32_t)__cvta_generic_to_shared(bars), sk = (uint32_t)__cvta_generic_to_shared(s_k), sv = (uint32_t)__cvta_generic_to_shared(s_v);
+    if (tid == 0) { mbar_init(bar, 1); mbar_init(bar + 8, 1); fence_mbar_init(); }
     if (!p.fused) { pdl_wait(); pdl_trigger(); }
     const uint32_t pos = __ldcg(a.pos) + t;                                              // a decode step's position was set before the step began
     const uint32_t n_seen = a.ring.active_len(pos + 1), lo = pos + 1 - n_seen;          // sinks are 0: the seen positions are consecutive
     const uint32_t per = (n_seen + cs - 1) / cs, j_lo = lo + min(n_seen, me * per), j_hi = lo + min(n_seen, (me + 1) * per);
-    if (p.fused) {
-        constexpr uint32_t LINES = D * sizeof(T) / 64;
-        for (uint32_t i = tid; i < (j_hi - j_lo) * LINES; i += RW_THREADS) {
-            const size_t at = (size_t)a.ring.slot_of_pos(j_lo + i / LINES) * D * sizeof(T) + (i % LINES) * 64;
-            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(kc) + at));
-            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(vc) + at));
-        }
-    }
+    // rows of positions j0 .. of one tile; a stale row of the new position may come along
+    auto request = [&](uint32_t dst, const T *cache, uint32_t j0, uint32_t b) {
+        const uint32_t n = min(TILE, j_hi - j0), slot = a.ring.slot_of_pos(j0), first = min(n, p.ring_rows - slot);
+        mbar_expect_tx(b, n * D * (uint32_t)sizeof(T));
+        bulk_g2s(dst, cache + (size_t)slot * D, first * D * (uint32_t)sizeof(T), b);
+        if (first < n) bulk_g2s(dst + first * D * (uint32_t)sizeof(T), cache, (n - first) * D * (uint32_t)sizeof(T), b);
+    };
+    auto landed = [&](uint32_t b, uint32_t parity) {
+        bool ok = false;
+        for (uint32_t spin = 0; spin < RW_WAIT_LIMIT && !ok; ++spin) ok = mbar_try_wait(b, parity);
+        if (!ok && a.err_flag != nullptr) atomicExch(a.err_flag, 1u);
+    };
+    if (tid == 0 && j_lo < j_hi) { request(sk, kc, j_lo, bar); request(sv, vc, j_lo, bar + 8); }
     for (uint32_t i = tid; i < gp * D; i += RW_THREADS) s_o[i] = 0.0f;
     for (uint32_t i = group * D + tid; i < gp * D; i += RW_THREADS) s_q[i] = 0.0f;
     for (uint32_t i = tid; i < gp; i += RW_THREADS) { s_m[i] = -INFINITY; s_l[i] = 0.0f; s_al[i] = 0.0f; }
+    const bool owner = p.fused && pos >= j_lo && pos < j_hi;          // this CTA attends to the new position and stores its rows
     if (p.fused) {
         pdl_wait();
         pdl_trigger();
         const float *x = a.qkv + t * a.qkv_stride;
-        for (uint32_t h = warp; h < group; h += RW_THREADS / 32) norm_row<float>(x + (g * group + h) * a.dim, a.q_norm, a.dim, D, a.eps, s_q + h * D, lane);
-        if (pos >= j_lo && pos < j_hi) {            // the CTA that attends to the new position stores its rows
-            const uint32_t slot = a.ring.slot_of_pos(pos);
-            if (warp == 7) norm_row<T>(x + (a.n_q + g) * a.dim, a.k_norm, a.dim, D, a.eps, kc + (size_t)slot * D, lane);
-            if (warp == 6) copy_row<T>(x + (a.n_q + a.n_kv) * a.dim + g * a.vdim, a.vdim, D, vc + (size_t)slot * D, lane);
+        for (uint32_t h = warp; h < group + (owner ? 2u : 0u); h += RW_THREADS / 32) {
+            if (h < group) norm_row<float>(x + (g * group + h) * a.dim, a.q_norm, a.dim, D, a.eps, s_q + h * D, lane);
+            else if (h == group) norm_row<float>(x + (a.n_q + g) * a.dim, a.k_norm, a.dim, D, a.eps, s_new, lane);
+            else copy_row<float>(x + (a.n_q + a.n_kv) * a.dim + g * a.vdim, a.vdim, D, s_new + D, lane);
         }
     } else {
         const T *qr = static_cast<const T *>(a.q) + ((size_t)t * a.n_q + g * group) * D;
@@ -132,23 +150,35 @@ __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams
         }
     }
     __syncthreads();
-    for (uint32_t j0 = j_lo; j0 < j_hi; j0 += RW_SC) {
-        const uint32_t n = min(RW_SC, j_hi - j0);
-        // scores: four lanes per key, sixteen keys per warp and step
+    if (owner) {
+        const size_t slot = (size_t)a.ring.slot_of_pos(pos) * D;
+        for (uint32_t i = tid; i < D; i += RW_THREADS) { put<T>(kc + slot + i, s_new[i]); put<T>(vc + slot + i, s_new[D + i]); }
+    }
+    uint32_t phase = 0;
+    for (uint32_t j0 = j_lo; j0 < j_hi; j0 += TILE, phase ^= 1) {
+        const uint32_t n = min(TILE, j_hi - j0), j_next = j0 + TILE;
+        const bool patch = owner && pos >= j0 && pos < j0 + n;
+        landed(bar, phase);
+        if (patch) {
+            for (uint32_t i = tid; i < D; i += RW_THREADS) put<T>(s_k + (pos - j0) * D + i, s_new[i]);
+            __syncthreads();
+        }
+        // scores: four lanes per key, sixteen keys per warp and step; neighbouring keys take their 64-byte pieces in another
+        // order, so that the eight lanes of a shared-memory phase hit different banks
         const uint32_t sub = lane & 3u, ki = lane >> 2;
 #pragma unroll 1
         for (uint32_t b = warp * 16; b < n; b += RW_THREADS / 2) {
             const uint32_t ja = b + ki, jb = b + 8 + ki;
-            const T *ka = kc + (size_t)a.ring.slot_of_pos(j0 + min(ja, n - 1)) * D, *kb = kc + (size_t)a.ring.slot_of_pos(j0 + min(jb, n - 1)) * D;
+            const T *ka = s_k + min(ja, n - 1) * D, *kb = s_k + min(jb, n - 1) * D;
 #pragma unroll 1
             for (uint32_t h0 = 0; h0 < group; h0 += HB) {
                 float da[HB], db[HB];
 #pragma unroll
                 for (uint32_t h = 0; h < HB; ++h) da[h] = db[h] = 0.0f;
-#pragma unroll
-                for (uint32_t c = 0; c < D / 32; ++c) {
+#pragma unroll 1
+                for (uint32_t c = 0; c < D / 32; ++c) {          // rolled: instruction fetch costs more than the loop
                     float va[8], vb[8];
-                    const uint32_t k = (c * 4 + sub) * 8;
+                    const uint32_t k = (((c + (ki & 1u)) % (D / 32)) * 4 + sub) * 8;
                     get8(ka + k, va);
                     get8(kb + k, vb);
 #pragma unroll
@@ -171,24 +201,28 @@ __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams
                     if (sub == (h & 3u)) {
                         const uint32_t hh = g * group + min(h0 + h, group - 1);
                         const float sc = __ldg(a.head_scale + hh), sl = __ldg(a.head_slope + hh);
-                        if (ja < n) s_p[(h0 + h) * RW_SC + ja] = da[h] * sc - sl * (float)(pos - (j0 + ja));
-                        if (jb < n) s_p[(h0 + h) * RW_SC + jb] = db[h] * sc - sl * (float)(pos - (j0 + jb));
+                        if (ja < n) s_p[(h0 + h) * TILE + ja] = da[h] * sc - sl * (float)(pos - (j0 + ja));
+                        if (jb < n) s_p[(h0 + h) * TILE + jb] = db[h] * sc - sl * (float)(pos - (j0 + jb));
                     }
             }
         }
         __syncthreads();
+        if (tid == 0 && j_next < j_hi) request(sk, kc, j_next, bar);         // everyone is done with the keys
 #pragma unroll 1
         for (uint32_t h = warp; h < group; h += RW_THREADS / 32) {          // softmax terms of the tile, one warp per head
             float mx = -INFINITY;
-            for (uint32_t j = lane; j < n; j += 32) mx = fmaxf(mx, s_p[h * RW_SC + j]);
+            for (uint32_t j = lane; j < n; j += 32) mx = fmaxf(mx, s_p[h * TILE + j]);
 #pragma unroll
             for (int m = 16; m > 0; m >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, m));
             const float m_old = s_m[h], m_new = fmaxf(m_old, mx);
             float sum = 0.0f;
-            for (uint32_t j = lane; j < n; j += 32) { const float e = expf(s_p[h * RW_SC + j] - m_new); s_p[h * RW_SC + j] = e; sum += e; }
+            for (uint32_t j = lane; j < n; j += 32) { const float e = expf(s_p[h * TILE + j] - m_new); s_p[h * TILE + j] = e; sum += e; }
             sum = warp_sum(sum);
             if (lane == 0) { const float al = expf(m_old - m_new); s_al[h] = al; s_m[h] = m_new; s_l[h] = s_l[h] * al + sum; }
         }
+        landed(bar + 8, phase);
+        if (patch)
+            for (uint32_t i = tid; i < D; i += RW_THREADS) put<T>(s_v + (pos - j0) * D + i, s_new[D + i]);
         __syncthreads();
         // values: thread = (key slice, eight columns); padding heads multiply finite leftovers that nobody reads
         constexpr uint32_t CPK = D / 8, KS = RW_THREADS / CPK;
@@ -201,13 +235,13 @@ __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams
 #pragma unroll
                 for (int i = 0; i < 8; ++i) acc[h][i] = 0.0f;
             if (ks < KS) {
-#pragma unroll 4
+#pragma unroll 2
                 for (uint32_t j = ks; j < n; j += KS) {
                     float v[8];
-                    get8(vc + (size_t)a.ring.slot_of_pos(j0 + j) * D + c * 8, v);
+                    get8(s_v + j * D + c * 8, v);
 #pragma unroll
                     for (uint32_t h = 0; h < HB; ++h) {
-                        const float e = s_p[(h0 + h) * RW_SC + j];
+                        const float e = s_p[(h0 + h) * TILE + j];
 #pragma unroll
                         for (int i = 0; i < 8; ++i) acc[h][i] = __fmaf_rn(e, v[i], acc[h][i]);
                     }
@@ -228,6 +262,7 @@ __global__ void __launch_bounds__(RW_THREADS) window_row_kernel(const AttnParams
             }
             __syncthreads();
         }
+        if (tid == 0 && j_next < j_hi) request(sv, vc, j_next, bar + 8);     // everyone is done with the values
     }
     // merge over the cluster: factors of every (head, CTA), then the outputs shared out over all CTAs
     __syncthreads();
@@ -427,7 +462,7 @@ cudaError_t row_launch_hb(cudaStream_t s, const AttnParams &p, int sm_count, boo
     uint32_t cs = 1;                            // CTAs per (token, kv head): at least 64 positions each, about one wave of CTAs
     const uint32_t longest = a.ring.window ? a.ring.window : p.ring_rows;
     while (cs < RW_MAX_CS && cs * 2 * 64 <= longest && cs * 2 * a.n_kv * p.n_tok <= (uint32_t)sm_count) cs *= 2;
-    const size_t smem = rw_smem(a.n_q / a.n_kv, D, HB);
+    const size_t smem = rw_smem<T>(a.n_q / a.n_kv, D, HB);
     cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(window_row_kernel<T, D, HB>), smem);
     if (e != cudaSuccess) return e;
     return launch_cluster(window_row_kernel<T, D, HB>, dim3(cs, a.n_kv, p.n_tok), dim3(RW_THREADS), smem, s, pdl, cs, p);
@@ -459,7 +494,7 @@ uint32_t window_attn_row(uint32_t dim, uint32_t vdim) {
     return 0;
 }
 
-bool window_attn_fits(bool f32, uint32_t group, uint32_t row) { return rw_smem(group, row, head_pass(f32, group)) <= 224 * 1024; }
+bool window_attn_fits(bool f32, uint32_t group, uint32_t row) { return (f32 ? rw_smem<float>(group, row, head_pass(f32, group)) : rw_smem<__nv_bfloat16>(group, row, head_pass(f32, group))) <= 224 * 1024; }
 
 cudaError_t launch_window_attention(cudaStream_t s, bool f32, const WindowAttnArgs &a, uint32_t n_tok, int sm_count, uint32_t *launches, bool pdl) {
     AttnParams p{a, n_tok, 0, n_tok == 1 ? 1u : 0u};
