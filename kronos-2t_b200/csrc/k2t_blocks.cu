@@ -284,7 +284,7 @@ extern "C" KronosCudaEngine *kronos_cuda_engine_create_blocks(KronosCudaContext 
     e->cfg.hidden_size = c.hidden_size; e->cfg.num_layers = c.num_blocks; e->cfg.vocab_size = c.vocab_size; e->cfg.max_seq_len = c.max_seq_len;
     e->cfg.rms_norm_eps = c.rms_norm_eps;
     e->layers.resize(n_blocks);
-    e->max_batch = 1024;                       // tokens per prompt batch: the row tiles of a projection times 256-token tiles fill the SMs
+    e->max_batch = 2048;                       // tokens per prompt batch: the row tiles of a projection times 256-token tiles fill the SMs
     if (const char *v = std::getenv("KRONOS_CUDA_PROMPT_BATCH")) e->max_batch = std::min(4096u, std::max(16u, ((uint32_t)std::strtoul(v, nullptr, 10) + 15u) & ~15u));
     e->max_batch = std::min(e->max_batch, std::max(16u, (c.max_seq_len + 15u) & ~15u));
     if (const char *v = std::getenv("KRONOS_CUDA_PDL")) e->pdl = v[0] != '0';
