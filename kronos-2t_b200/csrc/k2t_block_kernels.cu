@@ -21,8 +21,9 @@ __device__ __forceinline__ float4 load4(const float *p, uint32_t k, uint32_t n) 
 __device__ __forceinline__ float sq4(const float4 &v, float acc) {
     return __fmaf_rn(v.x, v.x, __fmaf_rn(v.y, v.y, __fmaf_rn(v.z, v.z, __fmaf_rn(v.w, v.w, acc))));
 }
+// z (1 + tanh(u)) / 2 = z / (1 + exp(-2 u)): the second form keeps its relative accuracy where tanh is near -1
 __device__ __forceinline__ float gelu_tanh(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
 template <bool F32>

@@ -62,6 +62,7 @@ ALONE = {
     "attention, one kv head, value size apart": [fm.attention(6, 1, 48, 80, 33)],
     "attention, as many kv heads, long rows": [fm.attention(3, 3, 136, 200, 70, scale=0.05)],
     "attention, large group": [fm.attention(20, 1, 16, 24, 50)],
+    "attention, itself only": [fm.attention(2, 1, 16, 16, 1)],
     "delta": [fm.delta(3, 32)],
     "delta, odd sizes": [fm.delta(2, 44, rank=70)],
     "delta, large head": [fm.delta(2, 128, rank=16)],
