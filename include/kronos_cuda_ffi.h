@@ -239,36 +239,63 @@ void kronos_cuda_engine_destroy(KronosCudaEngine *engine);
 
 /* ---- models described block by block (no counterpart in the reference) ---------------------------
  * Unquantized decoder models whose layers differ in kind: every block names its token mixer, its feed-forward (ff = 0: none)
- * and its sizes.  x += rms(mixer(x)) * norm1; with ff > 0: x += rms(down(act(up(x)))) * norm2; with side_dim > 0 the per-layer
- * token input x += rms(side_proj (gelu_tanh(side_gate x) * e)) * side_norm, e = the block's side_dim values of the token's row
- * of the side embedding table.  rms(v) = v / sqrt(mean(v^2) + rms_norm_eps).  All matrices are KRONOS_CUDA_MATRIX_DENSE with
- * bits = precision: 16 = bf16 products with fp32 accumulation (residual stream, norms, scores, softmax, recurrent state and
- * everything that enters a recurrence besides the products stay fp32), 32 = everything fp32.  Embedding tables are bf16. */
+ * and its sizes.  rms(v) = v / sqrt(mean(v^2) + rms_norm_eps), m = residual_mult:
+ *   x += m rms(mixer(pre1(x))) * norm1,   with ff > 0: x += m rms(ff(pre2(x))) * norm2,   pre(x) = rms(x) * pre_norm, or x without one
+ *   with side_dim > 0 the per-layer token input x += rms(side_proj (gelu_tanh(side_gate x) * e)) * side_norm, e = the block's
+ *   side_dim values of the token's row of the side embedding table (not together with pre-norms or residual_mult)
+ *   logits = head (rms(x) * final_norm), with logit_softcap > 0: cap tanh(logits / cap).
+ * All matrices are KRONOS_CUDA_MATRIX_DENSE with bits = precision: 16 = bf16 products with fp32 accumulation (residual stream,
+ * norms, scores, softmax, router scores, recurrent state and everything that enters a recurrence besides the products stay
+ * fp32), 32 = everything fp32.  Embedding tables are bf16. */
 #define KRONOS_CUDA_MIXER_WINDOW_ATTENTION 1u
 #define KRONOS_CUDA_MIXER_GENERAL_DELTA    2u
+#define KRONOS_CUDA_MIXER_LATENT_ATTENTION 3u
+
+/* Feed-forward: down act(up x).  POLYNORM: act = a N(z) + b N(z^2) + c N(z^3) + e with act_coef (not for experts); GELU_GATED: up_proj
+ * has 2 ff rows, 2i = gate i, 2i + 1 = up i, act = gelu_tanh(gate) * up; RELU_SQUARED: act = relu(z)^2. */
+#define KRONOS_CUDA_ACT_POLYNORM     0u
+#define KRONOS_CUDA_ACT_GELU_GATED   1u
+#define KRONOS_CUDA_ACT_RELU_SQUARED 2u
 
 typedef struct KronosCudaBlocksConfig {
     uint32_t struct_size;              /* sizeof(KronosCudaBlocksConfig), checked at creation */
     uint32_t hidden_size, num_blocks, vocab_size, max_seq_len, side_dim, precision;
     float rms_norm_eps;
+    float residual_mult;
+    float logit_softcap;               /* 0 = none */
 } KronosCudaBlocksConfig;
 
 typedef struct KronosCudaBlockDesc {
     uint32_t mixer, heads, kv_heads, dim, vdim;
-    uint32_t window;                   /* attention: position i sees 0 <= i - j < window; 0 = every earlier position */
+    uint32_t window;                   /* window attention: position i sees 0 <= i - j < window; 0 = every earlier position */
     uint32_t decay_rank, ff;
+    uint32_t q_rank, kv_rank, rot_dim; /* latent attention */
+    uint32_t act;                      /* KRONOS_CUDA_ACT_* */
+    /* experts > 0: ff is the size of one expert, each token takes the experts_top with the largest softmax scores (weights = the
+     * scores over all experts) and, with shared_ff > 0, an expert that serves every token with weight 1 */
+    uint32_t experts, experts_top, shared_ff;
     float decay_scale, unit_eps;       /* delta rule: w = exp(-decay_scale * sigmoid(.)), u = k / sqrt(sum k^2 + unit_eps) */
+    float score_scale;                 /* latent attention */
     const float *norm1, *norm2;        /* [hidden]; norm2 with ff > 0 */
-    /* attention: per-head RMS norm weights [dim]; score = (q . k) * head_scale[h] - head_slope[h] * (i - j), [heads] each */
+    const float *pre_norm1, *pre_norm2;        /* [hidden] or NULL */
+    /* window attention: per-head RMS norm weights [dim]; score = (q . k) * head_scale[h] - head_slope[h] * (i - j), [heads] each */
     const float *q_norm, *k_norm, *head_scale, *head_slope;
     /* delta rule, [heads * dim] each: decay = decay_proj tanh(.) + decay_bias, rate = sigmoid(. + rate_bias), norm weight of o */
     const float *decay_bias, *rate_bias, *out_norm;
-    const float *act_coef;             /* [4]: act = a N(z) + b N(z^2) + c N(z^3) + e, N = division by the rms over the ff values */
+    const float *act_coef;             /* POLYNORM: [4]; N = division by the rms over the ff values */
     const float *side_norm;            /* [hidden] */
-    /* attention: rows q (heads x dim), k (kv_heads x dim), v (kv_heads x vdim); o_proj [hidden][heads * vdim].
+    /* latent attention: norm weights of the latents [q_rank], [kv_rank]; (cos, sin) of the rotated pairs (2i, 2i + 1) at every position,
+     * [max_seq_len][rot_dim].  Blocks may share a table (it is copied once). */
+    const float *q_latent_norm, *kv_latent_norm, *rot_cos_sin;
+    /* window attention: rows q (heads x dim), k (kv_heads x dim), v (kv_heads x vdim); o_proj [hidden][heads * vdim].
      * delta rule: rows r, k, v, g, a (heads x dim each), then the decay_rank rows that feed tanh; decay_proj
-     * [heads * dim][decay_rank]; o_proj [hidden][heads * dim]. */
-    KronosCudaMatrixDesc in_proj, decay_proj, o_proj, up_proj, down_proj, side_gate, side_proj;
+     * [heads * dim][decay_rank]; o_proj [hidden][heads * dim].
+     * latent attention: rows query latent (q_rank), key/value latent (kv_rank), rotated key part (rot_dim); q_up
+     * [heads * (dim + rot_dim)][q_rank], per head dim plain and rot_dim rotated rows; kv_up [heads * (dim + vdim)][kv_rank], the keys of
+     * all heads, then the values; o_proj [hidden][heads * vdim].  score = (q . k + q_rot . k_rot) * score_scale.
+     * experts: up_proj and down_proj hold all experts one below the other, [experts * rows][..]; router [experts + rows of the shared
+     * expert's first product][hidden], the expert logits first; shared_down [hidden][shared_ff]. */
+    KronosCudaMatrixDesc in_proj, decay_proj, o_proj, up_proj, down_proj, side_gate, side_proj, q_up, kv_up, router, shared_down;
 } KronosCudaBlockDesc;
 
 /* The engine behind the handle is the one above: forward_token_ids, decode_greedy, profile_step, read_hidden, weight_bytes and

@@ -21,10 +21,6 @@ __device__ __forceinline__ float4 load4(const float *p, uint32_t k, uint32_t n) 
 __device__ __forceinline__ float sq4(const float4 &v, float acc) {
     return __fmaf_rn(v.x, v.x, __fmaf_rn(v.y, v.y, __fmaf_rn(v.z, v.z, __fmaf_rn(v.w, v.w, acc))));
 }
-// z (1 + tanh(u)) / 2 = z / (1 + exp(-2 u)): the second form keeps its relative accuracy where tanh is near -1
-__device__ __forceinline__ float gelu_tanh(float z) {
-    return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
-}
 
 template <bool F32>
 __global__ void __launch_bounds__(256) block_embed_kernel(const uint16_t *__restrict__ table, const uint32_t *__restrict__ tokens, uint32_t n, float *__restrict__ x,
@@ -38,32 +34,53 @@ __global__ void __launch_bounds__(256) block_embed_kernel(const uint16_t *__rest
     act_store<F32>(out, t, k, v);
 }
 
-template <bool F32, bool ADD>
-__global__ void __launch_bounds__(1024) block_norm_kernel(float *__restrict__ x, size_t x_stride, const float *__restrict__ y, size_t y_stride, const float *__restrict__ w,
-                                                         uint32_t n, float eps, const Act out) {
+template <bool F32, bool ADD, bool PRE>
+__global__ void __launch_bounds__(1024) block_norm_kernel(const NormArgs a) {
     __shared__ float scratch[32];
-    const uint32_t t = blockIdx.x;
-    float *xr = x + t * x_stride;
-    const float *src = ADD ? y + t * y_stride : xr;
+    const uint32_t t = blockIdx.x, n = a.n;
+    float *xr = a.x + t * a.x_stride, *yr = ADD ? a.y + t * a.y_stride : nullptr;
     pdl_wait();
     pdl_trigger();
-    float ss[1] = {0.0f};
-    const uint32_t step = blockDim.x * 4;
-    const uint32_t k_first = threadIdx.x * 4;
+    const uint32_t step = blockDim.x * 4, k_first = threadIdx.x * 4;
     float4 v0 = make_float4(0, 0, 0, 0), x0 = v0;          // the first step's values stay in registers
-    if (k_first < n) { v0 = load4(src, k_first, n); if (ADD) x0 = load4(xr, k_first, n); ss[0] = sq4(v0, ss[0]); }
-    for (uint32_t k = k_first + step; k < n; k += step) ss[0] = sq4(load4(src, k, n), ss[0]);
-    block_sum<1>(ss, scratch);
-    const float inv = 1.0f / sqrtf(ss[0] / (float)n + eps);
-    for (uint32_t k = k_first; k < n; k += step) {
-        const float4 v = k == k_first ? v0 : load4(src, k, n), g = __ldg(reinterpret_cast<const float4 *>(w + k));
-        float4 r = make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
-        if (ADD) {
-            const float4 o = k == k_first ? x0 : load4(xr, k, n);
-            r = make_float4(o.x + r.x, o.y + r.y, o.z + r.z, o.w + r.w);
+    float ss[1] = {0.0f};
+    if (ADD) {
+        auto sublayer = [&](uint32_t k) {
+            float4 v = load4(yr, k, n);
+            if (a.top > 0) {
+                for (uint32_t i = 0; i < a.top; ++i) {
+                    const float w = __ldcg(a.weight + t * a.top + i);
+                    const float4 q = load4(a.pairs + (size_t)__ldcg(a.row + t * a.top + i) * a.pair_stride, k, n);
+                    v = make_float4(__fmaf_rn(w, q.x, v.x), __fmaf_rn(w, q.y, v.y), __fmaf_rn(w, q.z, v.z), __fmaf_rn(w, q.w, v.w));
+                }
+                *reinterpret_cast<float4 *>(yr + k) = v;
+            }
+            return v;
+        };
+        if (k_first < n) { x0 = load4(xr, k_first, n); v0 = sublayer(k_first); ss[0] = sq4(v0, ss[0]); }
+        for (uint32_t k = k_first + step; k < n; k += step) ss[0] = sq4(sublayer(k), ss[0]);
+        block_sum<1>(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss[0] / (float)n + a.eps);
+        ss[0] = 0.0f;
+        for (uint32_t k = k_first; k < n; k += step) {
+            const float4 v = k == k_first ? v0 : load4(yr, k, n), o = k == k_first ? x0 : load4(xr, k, n), g = __ldg(reinterpret_cast<const float4 *>(a.post + k));
+            const float4 r = make_float4(o.x + a.mult * (v.x * inv * g.x), o.y + a.mult * (v.y * inv * g.y), o.z + a.mult * (v.z * inv * g.z), o.w + a.mult * (v.w * inv * g.w));
             *reinterpret_cast<float4 *>(xr + k) = r;
+            if (!PRE) act_store4<F32>(a.out, t, k, n, r);
+            if (PRE) ss[0] = sq4(r, ss[0]);
+            if (k == k_first) x0 = r;
         }
-        act_store4<F32>(out, t, k, n, r);
+    } else {
+        if (k_first < n) { x0 = load4(xr, k_first, n); ss[0] = sq4(x0, ss[0]); }
+        for (uint32_t k = k_first + step; k < n; k += step) ss[0] = sq4(load4(xr, k, n), ss[0]);
+    }
+    if (PRE) {
+        block_sum<1>(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss[0] / (float)n + a.eps);
+        for (uint32_t k = k_first; k < n; k += step) {
+            const float4 v = k == k_first ? x0 : load4(xr, k, n), g = __ldg(reinterpret_cast<const float4 *>(a.pre + k));
+            act_store4<F32>(a.out, t, k, n, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+        }
     }
 }
 
@@ -255,11 +272,12 @@ cudaError_t launch_block_embed(cudaStream_t s, bool f32, const uint16_t *table, 
     return launch_kernel(f32 ? block_embed_kernel<true> : block_embed_kernel<false>, dim3((n + 255) / 256, n_tok), dim3(256), 0, s, pdl, table, tokens, n, x, x_stride, out);
 }
 
-cudaError_t launch_block_norm(cudaStream_t s, bool f32, bool add, float *x, size_t x_stride, const float *y, size_t y_stride, const float *w, uint32_t n, float eps,
-                              const Act &out, uint32_t n_tok, bool pdl) {
-    const uint32_t threads = std::min(n_tok > 64 ? 512u : 1024u, std::max(32u, ((n + 3) / 4 + 31u) & ~31u));
-    auto k = f32 ? (add ? block_norm_kernel<true, true> : block_norm_kernel<true, false>) : (add ? block_norm_kernel<false, true> : block_norm_kernel<false, false>);
-    return launch_kernel(k, dim3(n_tok), dim3(threads), 0, s, pdl, x, x_stride, y, y_stride, w, n, eps, out);
+cudaError_t launch_block_norm(cudaStream_t s, bool f32, const NormArgs &a, uint32_t n_tok, bool pdl) {
+    if (a.y == nullptr && a.pre == nullptr) return cudaErrorInvalidValue;
+    const uint32_t threads = std::min(n_tok > 64 ? 512u : 1024u, std::max(32u, ((a.n + 3) / 4 + 31u) & ~31u));
+    auto k = f32 ? (a.y == nullptr ? block_norm_kernel<true, false, true> : a.pre == nullptr ? block_norm_kernel<true, true, false> : block_norm_kernel<true, true, true>)
+                 : (a.y == nullptr ? block_norm_kernel<false, false, true> : a.pre == nullptr ? block_norm_kernel<false, true, false> : block_norm_kernel<false, true, true>);
+    return launch_kernel(k, dim3(n_tok), dim3(threads), 0, s, pdl, a);
 }
 
 bool norm_side_fits(uint32_t n, uint32_t dim) { return ns_vec_smem(n, dim, 1) <= 200 * 1024; }

@@ -17,7 +17,7 @@ namespace {
 // (four with four CTAs per SM, six with two: more bytes in flight where the rows give only few CTAs).
 template <int NT, int GV_PF>
 __global__ void __launch_bounds__(256, NT == 1 && GV_PF == 4 ? 4 : 2) dense_gemv_kernel(const uint4 *__restrict__ w, uint32_t rows, uint32_t rows_pad, uint32_t np, const uint4 *__restrict__ x,
-                                                        uint32_t ld, uint32_t t0, uint32_t n_tok, float *__restrict__ out, size_t out_stride, uint32_t wk_log2) {
+                                                        uint32_t ld, uint32_t t0, uint32_t n_tok, const DenseOut out, uint32_t wk_log2) {
     __shared__ float s_part[8][8][NT];
     const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, wk = 1u << wk_log2, c = lane & 7u, r = lane >> 3;
     const uint32_t group = blockIdx.x * (8u >> wk_log2) + (warp >> wk_log2), ks = warp & (wk - 1);
@@ -75,14 +75,16 @@ __global__ void __launch_bounds__(256, NT == 1 && GV_PF == 4 ? 4 : 2) dense_gemv
         const uint32_t row_l = i & 7u, g = (i >> 3) % groups, t = (i >> 3) / groups;
         const uint32_t row = (blockIdx.x * groups + g) * 8 + row_l;
         if (row >= rows || t0 + t >= n_tok) continue;
-        float s = 0.0f;
+        float s = 0.0f, s1 = 0.0f;
         for (uint32_t k = 0; k < wk; ++k) s = __fadd_rn(s, s_part[g * wk + k][row_l][t]);
-        out[(size_t)(t0 + t) * out_stride + row] = s;
+        if (out.kind == Epi::GeluGated && (row_l & 1u) == 0)
+            for (uint32_t k = 0; k < wk; ++k) s1 = __fadd_rn(s1, s_part[g * wk + k][row_l + 1][t]);
+        dense_store<false>(out, t0 + t, row, s, s1);
     }
 }
 
 template <int NT>
-cudaError_t gemv_nt(cudaStream_t s, const DenseView &m, const Act &x, uint32_t t0, uint32_t n_tok, float *out, size_t out_stride, int sm_count, bool pdl) {
+cudaError_t gemv_nt(cudaStream_t s, const DenseView &m, const Act &x, uint32_t t0, uint32_t n_tok, const DenseOut &out, int sm_count, bool pdl) {
     const uint32_t groups = (m.rows + 7) / 8;
     // warps per row group: the fewest rounds of panels over the waves of the grid (a CTA beyond a full wave costs a whole round)
     const uint32_t slots = (uint32_t)sm_count * (NT == 1 ? 4u : 2u);
@@ -97,7 +99,7 @@ cudaError_t gemv_nt(cudaStream_t s, const DenseView &m, const Act &x, uint32_t t
     const uint32_t per = 8u >> wl, ctas = (groups + per - 1) / per;
     auto k = NT == 1 && ctas <= 2u * (uint32_t)sm_count ? dense_gemv_kernel<NT, NT == 1 ? 6 : 4> : dense_gemv_kernel<NT, 4>;
     return launch_kernel(k, dim3(ctas), dim3(256), 0, s, pdl, static_cast<const uint4 *>(m.base), m.rows, m.rows_pad, m.panels,
-                         static_cast<const uint4 *>(x.p), x.ld, t0, n_tok, out, out_stride, wl);
+                         static_cast<const uint4 *>(x.p), x.ld, t0, n_tok, out, wl);
 }
 
 // ------------------------------------------------------------------------------------------------ bf16 GEMM (tensor cores)
@@ -115,9 +117,11 @@ template <int NT> __host__ __device__ constexpr uint32_t gm_smem() { return GM_H
 struct GemmArgs {
     const uint8_t *w, *x;
     uint32_t rows, rows_pad, np, ld, n_tok;
-    float *out;
-    size_t out_stride;
+    DenseOut out;
     uint32_t *err_flag;
+    const void *const *bases;           // GROUPED: images of the experts, blockIdx.y = item
+    const ExpertItem *items;
+    const uint32_t *n_items;
 };
 
 __device__ __forceinline__ bool gm_wait(uint32_t bar, uint32_t parity, volatile uint32_t *abort_w) {
@@ -153,12 +157,53 @@ __device__ __forceinline__ void gm_ld32(uint32_t taddr, uint32_t (&v)[32]) {
         : "r"(taddr) : "memory");
 }
 
-template <int NT>
+// 32 sums per lane (lane = row, registers = tokens tok .. tok + n - 1) -> output.  Activations: neighbouring lanes swap halves, so
+// that a lane stores two columns (or one product of a pair) of every second token.
+__device__ __forceinline__ void gm_store(const DenseOut &o, uint32_t rows, uint32_t row, uint32_t tok, uint32_t n, uint32_t (&v)[32]) {
+    if (o.kind == Epi::Rows || o.kind == Epi::Softcap) {
+        if (row >= rows) return;
+        float *p = o.rows + (size_t)tok * o.stride + row;
+#pragma unroll
+        for (uint32_t t = 0; t < 32; ++t) {
+            float x = __uint_as_float(v[t]);
+            if (o.kind == Epi::Softcap) x = softcap(x, o.cap);
+            if (t < n) p[t * o.stride] = x;
+        }
+        return;
+    }
+    const bool odd = (threadIdx.x & 1u) != 0;
+#pragma unroll
+    for (uint32_t t = 0; t < 32; t += 2) {
+        const float mine = __uint_as_float(odd ? v[t + 1] : v[t]), other = __shfl_xor_sync(0xffffffffu, __uint_as_float(odd ? v[t] : v[t + 1]), 1);
+        const uint32_t tt = t + (odd ? 1u : 0u), r = row & ~1u;
+        const float lo = odd ? other : mine, hi = odd ? mine : other;       // rows r and r + 1 of token tt
+        if (tt >= n || r >= rows) continue;
+        if (o.kind == Epi::GeluGated) {
+            act_store<false>(o.act, tok + tt, r >> 1, gelu_tanh(lo) * hi);
+        } else {
+            const float x = o.kind == Epi::Relu2 ? relu_squared(lo) : lo, y = o.kind == Epi::Relu2 ? relu_squared(hi) : hi;
+            if (r + 1 < rows) *reinterpret_cast<uint32_t *>(static_cast<__nv_bfloat16 *>(o.act.p) + panel_index(o.act.ld, tok + tt, r)) = pack_bf16(x, y);
+            else act_store<false>(o.act, tok + tt, r, x);
+        }
+    }
+}
+
+template <int NT, bool GROUPED>
 __global__ void __launch_bounds__(GM_THREADS) dense_gemm_kernel(const GemmArgs a) {
     extern __shared__ uint8_t smem_raw[];
     constexpr uint32_t S = gm_stages<NT>(), B_BYTES = NT * PANEL * 2;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const uint32_t row0 = blockIdx.x * DENSE_ROW_TILE, tok0 = blockIdx.y * NT;
+    const uint32_t row0 = blockIdx.x * DENSE_ROW_TILE;
+    uint32_t tok0 = blockIdx.y * NT, tok_end = a.n_tok;
+    const uint8_t *w = a.w;
+    if (GROUPED) {                       // the items come from the predecessor
+        pdl_wait();
+        if (blockIdx.y >= __ldcg(a.n_items)) return;
+        const ExpertItem it = a.items[blockIdx.y];
+        tok0 = it.row0;
+        tok_end = it.row_end;
+        w = static_cast<const uint8_t *>(a.bases[it.expert]);
+    }
     const uint32_t raw = (uint32_t)__cvta_generic_to_shared(smem_raw), sbase = (raw + 1023u) & ~1023u;
     uint8_t *smem = smem_raw + (sbase - raw);
     const uint32_t bar_full = sbase, bar_empty = sbase + 64, bar_done = sbase + 128;
@@ -182,7 +227,7 @@ __global__ void __launch_bounds__(GM_THREADS) dense_gemm_kernel(const GemmArgs a
 
     if (warp == 4) {
         if (lane == 0) {
-            const uint8_t *wsrc = a.w + (size_t)row0 * (PANEL * 2), *xsrc = a.x + (size_t)tok0 * (PANEL * 2);
+            const uint8_t *wsrc = w + (size_t)row0 * (PANEL * 2), *xsrc = a.x + (size_t)tok0 * (PANEL * 2);
             const size_t w_pitch = (size_t)a.rows_pad * (PANEL * 2), x_pitch = (size_t)a.ld * (PANEL * 2);
             const uint32_t pre = min(S, a.np);
             for (uint32_t p = 0; p < pre; ++p) {            // the weights do not depend on the predecessor
@@ -237,16 +282,10 @@ __global__ void __launch_bounds__(GM_THREADS) dense_gemm_kernel(const GemmArgs a
         const uint32_t row = row0 + warp * 32 + lane;
 #pragma unroll 1
         for (uint32_t c = 0; c < NT; c += 32) {
-            if (tok0 + c >= a.n_tok || !ok) break;
+            if (tok0 + c >= tok_end || !ok) break;
             uint32_t v[32];
             gm_ld32(tmem + ((warp * 32u) << 16) + c, v);
-            if (row < a.rows) {
-                float *o = a.out + (size_t)(tok0 + c) * a.out_stride + row;
-                const uint32_t n = min(32u, a.n_tok - tok0 - c);
-#pragma unroll
-                for (uint32_t t = 0; t < 32; ++t)
-                    if (t < n) o[t * a.out_stride] = __uint_as_float(v[t]);
-            }
+            gm_store(a.out, a.rows, row, tok0 + c, min(32u, tok_end - tok0 - c), v);
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -258,9 +297,9 @@ __global__ void __launch_bounds__(GM_THREADS) dense_gemm_kernel(const GemmArgs a
 }
 
 template <int NT> cudaError_t gemm_nt(cudaStream_t s, const GemmArgs &a, bool pdl) {
-    cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(dense_gemm_kernel<NT>), gm_smem<NT>());
+    cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(dense_gemm_kernel<NT, false>), gm_smem<NT>());
     if (e != cudaSuccess) return e;
-    return launch_kernel(dense_gemm_kernel<NT>, dim3(a.rows_pad / DENSE_ROW_TILE, (a.n_tok + NT - 1) / NT), dim3(GM_THREADS), gm_smem<NT>(), s, pdl, a);
+    return launch_kernel(dense_gemm_kernel<NT, false>, dim3(a.rows_pad / DENSE_ROW_TILE, (a.n_tok + NT - 1) / NT), dim3(GM_THREADS), gm_smem<NT>(), s, pdl, a);
 }
 
 // ------------------------------------------------------------------------------------------------ fp32
@@ -329,6 +368,16 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const float *__rest
     }
 }
 
+__global__ void __launch_bounds__(256) dense_epilogue_f32_kernel(uint32_t rows, uint32_t n_tok, const DenseOut out) {
+    pdl_wait();
+    pdl_trigger();
+    for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < (size_t)n_tok * rows; i += (size_t)gridDim.x * 256) {
+        const uint32_t t = (uint32_t)(i / rows), r = (uint32_t)(i % rows);
+        const float *p = out.rows + (size_t)t * out.stride + r;
+        dense_store<true>(out, t, r, *p, out.kind == Epi::GeluGated && r + 1 < rows ? p[1] : 0.0f);
+    }
+}
+
 template <bool F32>
 __global__ void __launch_bounds__(256) dense_pack_kernel(const float *__restrict__ x, uint32_t n_tok, uint32_t cols, uint32_t padded, const Act out) {
     pdl_wait();
@@ -347,21 +396,22 @@ cudaError_t launch_dense_pack(cudaStream_t s, bool f32, const float *x, uint32_t
     return launch_kernel(f32 ? dense_pack_kernel<true> : dense_pack_kernel<false>, dim3(ctas), dim3(256), 0, s, pdl, x, n_tok, cols, padded, out);
 }
 
-cudaError_t launch_dense(cudaStream_t s, const DeviceMatrix &dm, const Act &x, uint32_t n_tok, float *out, size_t out_stride, int sm_count,
-                         uint32_t *err_flag, uint32_t *launches, bool pdl) {
+cudaError_t launch_dense_out(cudaStream_t s, const DeviceMatrix &dm, const Act &x, uint32_t n_tok, const DenseOut &out, int sm_count, uint32_t *err_flag,
+                             uint32_t *launches, bool pdl) {
     const DenseView m = dense_view(dm);
     *launches = 0;
     if (n_tok == 0) return cudaSuccess;
     if (dm.geom.fmt == FMT_DENSE32) {
-        *launches = 1;
+        *launches = out.kind == Epi::Rows ? 1 : 2;
         const float *w = static_cast<const float *>(m.base), *xv = static_cast<const float *>(x.p);
-        if (n_tok < 16)
-            return launch_kernel(dense_gemv_f32_kernel<4>, dim3((m.rows + 7) / 8, (n_tok + 3) / 4), dim3(256), 0, s, pdl, w, m.rows, m.rows_pad, xv, x.ld, n_tok, out, out_stride);
-        return launch_kernel(dense_gemm_f32_kernel, dim3((m.rows + 63) / 64, (n_tok + 63) / 64), dim3(256), 0, s, pdl, w, m.rows, m.rows_pad, xv, x.ld, n_tok, out, out_stride);
+        const cudaError_t e = n_tok < 16 ? launch_kernel(dense_gemv_f32_kernel<4>, dim3((m.rows + 7) / 8, (n_tok + 3) / 4), dim3(256), 0, s, pdl, w, m.rows, m.rows_pad, xv, x.ld, n_tok, out.rows, out.stride)
+                                         : launch_kernel(dense_gemm_f32_kernel, dim3((m.rows + 63) / 64, (n_tok + 63) / 64), dim3(256), 0, s, pdl, w, m.rows, m.rows_pad, xv, x.ld, n_tok, out.rows, out.stride);
+        if (e != cudaSuccess || out.kind == Epi::Rows) return e;
+        return launch_kernel(dense_epilogue_f32_kernel, dim3((uint32_t)std::min<size_t>(1184, ((size_t)n_tok * m.rows + 255) / 256)), dim3(256), 0, s, pdl, m.rows, n_tok, out);
     }
     if (dm.geom.fmt != FMT_DENSE16) return cudaErrorInvalidValue;
     if (n_tok >= DENSE_TC_MIN) {
-        const GemmArgs a{static_cast<const uint8_t *>(m.base), static_cast<const uint8_t *>(x.p), m.rows, m.rows_pad, m.panels, x.ld, n_tok, out, out_stride, err_flag};
+        const GemmArgs a{static_cast<const uint8_t *>(m.base), static_cast<const uint8_t *>(x.p), m.rows, m.rows_pad, m.panels, x.ld, n_tok, out, err_flag, nullptr, nullptr, nullptr};
         // widest token tile that does not leave SMs idle: relative time of a tile against the waves of the grid
         static const struct { uint32_t nt; float cost; } tiles[4] = {{256, 1.0f}, {128, 0.55f}, {64, 0.34f}, {32, 0.25f}};
         uint32_t best = 32;
@@ -377,12 +427,22 @@ cudaError_t launch_dense(cudaStream_t s, const DeviceMatrix &dm, const Act &x, u
     // weight passes of up to eight tokens (rows of the activation are padded to eight: a pass may read, never store, beyond n_tok)
     for (uint32_t t0 = 0; t0 < n_tok; t0 += 8) {
         const uint32_t left = n_tok - t0;
-        const cudaError_t e = left > 4 ? gemv_nt<8>(s, m, x, t0, n_tok, out, out_stride, sm_count, pdl) : left > 2 ? gemv_nt<4>(s, m, x, t0, n_tok, out, out_stride, sm_count, pdl)
-                              : left == 2 ? gemv_nt<2>(s, m, x, t0, n_tok, out, out_stride, sm_count, pdl) : gemv_nt<1>(s, m, x, t0, n_tok, out, out_stride, sm_count, pdl);
+        const cudaError_t e = left > 4 ? gemv_nt<8>(s, m, x, t0, n_tok, out, sm_count, pdl) : left > 2 ? gemv_nt<4>(s, m, x, t0, n_tok, out, sm_count, pdl)
+                              : left == 2 ? gemv_nt<2>(s, m, x, t0, n_tok, out, sm_count, pdl) : gemv_nt<1>(s, m, x, t0, n_tok, out, sm_count, pdl);
         *launches += 1;
         if (e != cudaSuccess) return e;
     }
     return cudaSuccess;
+}
+
+cudaError_t launch_dense_experts(cudaStream_t s, const ExpertView &m, const Act &x, const ExpertItem *items, const uint32_t *n_items, uint32_t max_items,
+                                 const DenseOut &out, uint32_t *err_flag, bool pdl) {
+    if (max_items == 0 || max_items > 65535u) return cudaErrorInvalidValue;
+    constexpr int NT = (int)EXPERT_TILE;
+    const GemmArgs a{nullptr, static_cast<const uint8_t *>(x.p), m.rows, m.rows_pad, m.panels, x.ld, 0u, out, err_flag, m.base, items, n_items};
+    cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(dense_gemm_kernel<NT, true>), gm_smem<NT>());
+    if (e != cudaSuccess) return e;
+    return launch_kernel(dense_gemm_kernel<NT, true>, dim3(m.rows_pad / DENSE_ROW_TILE, max_items), dim3(GM_THREADS), gm_smem<NT>(), s, pdl, a);
 }
 
 }  // namespace k2t

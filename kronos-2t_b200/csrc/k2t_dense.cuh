@@ -62,6 +62,25 @@ template <bool F32, bool SHARED = false> __device__ __forceinline__ float row_do
     return acc;
 }
 
+// z (1 + tanh(u)) / 2 = z / (1 + exp(-2 u)): the second form keeps its relative accuracy where tanh is near -1
+__device__ __forceinline__ float gelu_tanh(float z) {
+    return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float relu_squared(float z) { const float r = fmaxf(z, 0.0f); return r * r; }
+__device__ __forceinline__ float softcap(float z, float cap) { return cap * tanhf(z / cap); }
+// sum of row r (and, for pairs, of row r + 1 behind an even r) of token t -> output
+template <bool F32> __device__ __forceinline__ void dense_store(const DenseOut &o, uint32_t t, uint32_t r, float v, float next) {
+    switch (o.kind) {
+        case Epi::Rows: o.rows[(size_t)t * o.stride + r] = v; break;
+        case Epi::Softcap: o.rows[(size_t)t * o.stride + r] = softcap(v, o.cap); break;
+        case Epi::Panels: act_store<F32>(o.act, t, r, v); break;
+        case Epi::Relu2: act_store<F32>(o.act, t, r, relu_squared(v)); break;
+        case Epi::GeluGated:
+            if ((r & 1u) == 0) act_store<F32>(o.act, t, r >> 1, gelu_tanh(v) * next);
+            break;
+    }
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int m = 16; m > 0; m >>= 1) v = __fadd_rn(v, __shfl_xor_sync(0xffffffffu, v, m));

@@ -43,12 +43,46 @@ inline DenseView dense_view(const DeviceMatrix &m) {
     return DenseView{m.d_base, m.geom.rows, m.geom.cols, m.geom.fmt == FMT_DENSE32 ? dense_f32_ld(m.geom.cols) : m.geom.rows_pad, m.geom.nc};
 }
 
-// out[t * out_stride + r] = sum over k of W[r][k] x[t][k], fp32 accumulation.  bf16: up to DENSE_TC_MIN - 1 tokens as weight
-// passes of up to eight tokens, more on the tensor cores; fp32: plain fused multiply-adds.
+// What becomes of the sums out[t][r] = sum over k of W[r][k] x[t][k] (fp32 accumulation).
+enum class Epi : uint32_t {
+    Rows,           // fp32 rows
+    Softcap,        // fp32 rows of cap * tanh(sum / cap)
+    Panels,         // activation of another product, column r
+    Relu2,          // activation of relu(sum)^2
+    GeluGated,      // rows come in pairs (gate i, up i): activation of gelu_tanh(gate) * up, column i
+};
+struct DenseOut {
+    Epi kind;
+    float *rows;                            // Rows, Softcap; scratch for the others where the matrix is fp32
+    size_t stride;
+    float cap;
+    Act act;
+};
+inline DenseOut dense_rows(float *out, size_t stride) { return DenseOut{Epi::Rows, out, stride, 0.0f, Act{}}; }
+
+// bf16: up to DENSE_TC_MIN - 1 tokens as weight passes of up to eight tokens, more on the tensor cores; fp32: plain fused
+// multiply-adds, activations by a second kernel.
 constexpr uint32_t DENSE_TC_MIN = 17;
-cudaError_t launch_dense(cudaStream_t s, const DeviceMatrix &m, const Act &x, uint32_t n_tok, float *out, size_t out_stride, int sm_count,
-                         uint32_t *err_flag, uint32_t *launches, bool pdl);
+cudaError_t launch_dense_out(cudaStream_t s, const DeviceMatrix &m, const Act &x, uint32_t n_tok, const DenseOut &out, int sm_count, uint32_t *err_flag,
+                             uint32_t *launches, bool pdl);
+inline cudaError_t launch_dense(cudaStream_t s, const DeviceMatrix &m, const Act &x, uint32_t n_tok, float *out, size_t out_stride, int sm_count,
+                                uint32_t *err_flag, uint32_t *launches, bool pdl) {
+    return launch_dense_out(s, m, x, n_tok, dense_rows(out, out_stride), sm_count, err_flag, launches, pdl);
+}
 // fp32 rows [n_tok][cols] -> activation
 cudaError_t launch_dense_pack(cudaStream_t s, bool f32, const float *x, uint32_t n_tok, uint32_t cols, const Act &out, bool pdl);
+
+// ---- one matrix per expert (all of one shape): device table of their images
+struct ExpertView {
+    const void *const *base;
+    uint32_t rows, cols, rows_pad, panels;  // of one expert, see DenseView
+};
+// A stretch of rows [row0, row_end) of a packed activation that one expert works on; row0 is a multiple of eight.
+struct ExpertItem { uint32_t expert, row0, row_end, pad; };
+constexpr uint32_t EXPERT_TILE = 64;        // rows of the packed activation per item
+// tensor-core product of every item's rows with its expert; items and their number live on the device (at most max_items).
+// Row p of the packed activation gives row p of the output.
+cudaError_t launch_dense_experts(cudaStream_t s, const ExpertView &m, const Act &x, const ExpertItem *items, const uint32_t *n_items, uint32_t max_items,
+                                 const DenseOut &out, uint32_t *err_flag, bool pdl);
 
 }  // namespace k2t

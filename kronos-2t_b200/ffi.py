@@ -53,20 +53,22 @@ class LayerDesc(C.Structure):
                 ("moe_shared_gate_w", C.c_void_p)]
 
 
-MIXER_WINDOW_ATTENTION, MIXER_GENERAL_DELTA = 1, 2
+MIXER_WINDOW_ATTENTION, MIXER_GENERAL_DELTA, MIXER_LATENT_ATTENTION = 1, 2, 3
+ACT_POLYNORM, ACT_GELU_GATED, ACT_RELU_SQUARED = 0, 1, 2
 
 
 class BlocksConfig(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("struct_size", "hidden_size", "num_blocks", "vocab_size", "max_seq_len", "side_dim", "precision")] + \
-               [("rms_norm_eps", C.c_float)]
+               [(n, C.c_float) for n in ("rms_norm_eps", "residual_mult", "logit_softcap")]
 
 
 class BlockDesc(C.Structure):
-    _fields_ = [(n, C.c_uint32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "window", "decay_rank", "ff")] + \
-               [("decay_scale", C.c_float), ("unit_eps", C.c_float)] + \
-               [(n, C.c_void_p) for n in ("norm1", "norm2", "q_norm", "k_norm", "head_scale", "head_slope", "decay_bias", "rate_bias", "out_norm",
-                                          "act_coef", "side_norm")] + \
-               [(n, MatrixDesc) for n in ("in_proj", "decay_proj", "o_proj", "up_proj", "down_proj", "side_gate", "side_proj")]
+    _fields_ = [(n, C.c_uint32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "window", "decay_rank", "ff", "q_rank", "kv_rank", "rot_dim", "act",
+                                          "experts", "experts_top", "shared_ff")] + \
+               [(n, C.c_float) for n in ("decay_scale", "unit_eps", "score_scale")] + \
+               [(n, C.c_void_p) for n in ("norm1", "norm2", "pre_norm1", "pre_norm2", "q_norm", "k_norm", "head_scale", "head_slope", "decay_bias", "rate_bias", "out_norm",
+                                          "act_coef", "side_norm", "q_latent_norm", "kv_latent_norm", "rot_cos_sin")] + \
+               [(n, MatrixDesc) for n in ("in_proj", "decay_proj", "o_proj", "up_proj", "down_proj", "side_gate", "side_proj", "q_up", "kv_up", "router", "shared_down")]
 
 
 def load_library():
@@ -425,7 +427,8 @@ class Engine:
 
     def _create_blocks(self, spec):
         c, keep = spec["cfg"], []
-        self.cfg = BlocksConfig(C.sizeof(BlocksConfig), c["hidden"], len(spec["blocks"]), c["vocab"], c["max_seq"], c.get("side_dim", 0), c["precision"], c["eps"])
+        self.cfg = BlocksConfig(C.sizeof(BlocksConfig), c["hidden"], len(spec["blocks"]), c["vocab"], c["max_seq"], c.get("side_dim", 0), c["precision"], c["eps"],
+                                c.get("residual_mult", 1.0), c.get("logit_softcap", 0.0))
         self.vocab = c["vocab"]
 
         def fill(d, field, value):

@@ -4,8 +4,8 @@
     spec = load_spec(folder, dtype="bfloat16", max_seq=4096)
     engine = load_engine(ctx, folder)
 
-Registered: `Folizen` (config.json + model.safetensors: blocks of sliding-window attention and generalized delta rule), and the
-compiled Llama / Qwen models (a Hugging Face config.json beside one .k2tb container)."""
+Registered: `Folizen` (config.json + model.safetensors: blocks of sliding-window attention and generalized delta rule), `Zasesun`
+(the same files: blocks of latent attention, dense or expert feed-forwards), and the compiled Llama / Qwen models (a Hugging Face config.json beside one .k2tb container)."""
 import glob
 import json
 import mmap
@@ -138,6 +138,78 @@ def folizen_spec(folder, config, dtype, max_seq):
     vocab, width = t.shape("embed")
     return dict(cfg=dict(hidden=width, vocab=vocab, max_seq=max_seq, eps=config["norm"]["eps"], side_dim=side, precision=16 if dtype == "bfloat16" else 32),
                 blocks=blocks, final_norm=t.f32("final.norm"), head=mat("head"), embed=t.bits("embed"), side_embed=t.bits("side.embed") if side else None)
+
+
+# ---- rotary positions
+def yarn_frequencies(dims, base, scaling=None):
+    """(frequency of every rotated pair, factor of cos and sin), float64.  scaling {factor, original, fast, slow}: pairs that turn more
+    than `fast` times within `original` positions keep their frequency, those that turn less than `slow` times have it divided by
+    `factor`, with a linear ramp over the pairs in between."""
+    i = np.arange(dims // 2)
+    freq = float(base) ** (-2.0 * i / dims)
+    if not scaling:
+        return freq, 1.0
+    pair = lambda turns: dims * np.log(scaling["original"] / (2.0 * np.pi * turns)) / (2.0 * np.log(base))
+    lo, hi = max(np.floor(pair(scaling["fast"])), 0), min(np.ceil(pair(scaling["slow"])), dims - 1)
+    ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return freq / scaling["factor"] * ramp + freq * (1.0 - ramp), 0.1 * np.log(scaling["factor"]) + 1.0
+
+
+def rotation_table(positions, width, dims, base, scaling=None):
+    """[positions][width]: (cos, sin) of every neighbouring pair; pairs from `dims` on stay as they are."""
+    freq, gain = yarn_frequencies(dims, base, scaling)
+    angle = np.arange(positions)[:, None] * freq
+    table = np.zeros((positions, width), np.float32)
+    table[:, 0::2] = 1.0
+    table[:, 0:dims:2], table[:, 1:dims:2] = np.cos(angle) * gain, np.sin(angle) * gain
+    return table
+
+
+# ---- Zasesun
+@register("Zasesun")
+def zasesun_spec(folder, config, dtype, max_seq):
+    t = Tensors(os.path.join(folder, "model.safetensors"))
+    mat = t.bits if dtype == "bfloat16" else t.f32
+    tables = {}
+
+    def rows(*names):
+        return np.concatenate([mat(n) for n in names])
+
+    blocks = []
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        x = p + "mix."
+        if layer["type"] != "latent_attention":
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        rot = m["rot"]
+        key = json.dumps([m["rot_dim"], rot], sort_keys=True)
+        if key not in tables:
+            tables[key] = rotation_table(max_seq, m["rot_dim"], rot["dims"], rot["base"], rot.get("scaling"))
+        b = dict(mixer=ffi.MIXER_LATENT_ATTENTION, heads=m["heads"], dim=m["dim"], vdim=m["vdim"], rot_dim=m["rot_dim"], kv_rank=m["kv_rank"],
+                 q_rank=t.shape(x + "dq")[0], score_scale=m["scale"], rot_cos_sin=tables[key], q_latent_norm=t.f32(x + "dq.norm"),
+                 kv_latent_norm=t.f32(x + "dkv.norm"), pre_norm1=t.f32(p + "norm1"), norm1=t.f32(p + "norm1b"),
+                 in_proj=rows(x + "dq", x + "dkv"), q_up=mat(x + "uq"), kv_up=rows(x + "uk", x + "uv"), o_proj=mat(x + "o"))
+        mlp, f = layer.get("mlp"), p + "mlp."
+        if mlp is not None:
+            b.update(pre_norm2=t.f32(p + "norm2"), norm2=t.f32(p + "norm2b"))
+            kind = mlp.get("kind", "dense")
+            if kind == "dense":
+                gate, up = mat(f + "gate"), mat(f + "up")
+                b.update(act=ffi.ACT_GELU_GATED, ff=up.shape[0], up_proj=np.stack([gate, up], 1).reshape(-1, up.shape[1]), down_proj=mat(f + "down"))
+            elif kind == "moe":
+                n, shared = mlp["router"]["experts"], mlp.get("shared") is not None
+                b.update(act=ffi.ACT_RELU_SQUARED, experts=n, experts_top=mlp["router"]["top"], ff=t.shape(f + "e0.up")[0],
+                         up_proj=rows(*(f"{f}e{e}.up" for e in range(n))), down_proj=rows(*(f"{f}e{e}.down" for e in range(n))),
+                         router=rows(f + "router", *([f + "shared.up"] if shared else [])))
+                if shared:
+                    b.update(shared_ff=t.shape(f + "shared.up")[0], shared_down=mat(f + "shared.down"))
+            else:
+                raise ValueError(f"layer {i}: unknown feed-forward {kind!r}")
+        blocks.append(b)
+    embed = mat("embed")
+    return dict(cfg=dict(hidden=embed.shape[1], vocab=embed.shape[0], max_seq=max_seq, eps=config["norm"]["eps"], residual_mult=config["residual_mult"],
+                         logit_softcap=config["logit_softcap"], precision=16 if dtype == "bfloat16" else 32),
+                blocks=blocks, final_norm=t.f32("final.norm"), head=embed, embed=t.bits("embed"))
 
 
 # ---- compiled Llama / Qwen models
