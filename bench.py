@@ -938,9 +938,29 @@ def _folizen_flops(c, n_layers):
     return 2 * ((n_layers + 1) // 2 * attn + n_layers // 2 * delta)
 
 
-def run_folizen(args, local_rank):
-    """Block models (random bf16 weights): prompt and decode throughput at real layer sizes, beside a Llama shape of the same
-    width, depth, heads and MLP on the quantized engine (nf4g128 weights, int8 cache)."""
+def _zasesun_bytes(c, n_layers, ctx_len):
+    """(weight bytes, latent cache bytes) one decoded token streams (the experts it takes, not all)."""
+    h, H = c["hidden"], c["heads"]
+    attn = (c["q_rank"] + c["kv_rank"] + c["rot_dim"]) * h + H * (c["dim"] + c["rot_dim"]) * c["q_rank"] + H * (c["dim"] + c["vdim"]) * c["kv_rank"] + h * H * c["vdim"]
+    dense, moe = 3 * c["ff"] * h, (c["experts"] + 2 * c["shared_ff"] + 2 * c["top"] * c["expert_ff"]) * h
+    return 2 * (n_layers * attn + (n_layers + 1) // 2 * dense + n_layers // 2 * moe + c["vocab"] * h), n_layers * ctx_len * (c["kv_rank"] + c["rot_dim"]) * 2
+
+
+def _attention_like_bytes(c, n_layers, ctx_len):
+    h, hd, kv = c["hidden"], c["heads"] * c["dim"], c["kv_heads"] * c["dim"]
+    ffs = [c["ff_turns"][i % 2] for i in range(n_layers)]
+    return 2 * (n_layers * ((hd + 2 * kv) * h + h * hd) + sum(2 * f * h for f in ffs) + c["vocab"] * h), n_layers * 2 * ctx_len * kv * 2
+
+
+def _product_flops(weight_bytes, c):
+    """2 x multiply-adds of one prompt token's products (head left out)."""
+    return weight_bytes - 2 * c["vocab"] * c["hidden"]
+
+
+def run_block_models(args, local_rank, design):
+    """Block models (random bf16 weights): prompt and decode throughput at real layer sizes.  folizen: beside a Llama shape of the same
+    width, depth, heads and MLP on the quantized engine (nf4g128 weights, int8 cache); zasesun: beside a Folizen shape (attention
+    over every position) of the same width, depth, heads and active feed-forward size."""
     import numpy as np
     import torch
     import kronos_2t_b200 as k2
@@ -968,28 +988,44 @@ def run_folizen(args, local_rank):
             best = e0.elapsed_time(e1) if best is None else min(best, e0.elapsed_time(e1))
         return best
 
-    out = {"mode": "folizen", "peak_kind": peak_kind, "data": "synthetic (random weights)", "models": []}
-    steps = args.folizen_steps
+    sizes, shapes = (args.folizen, synth.FOLIZEN_SHAPES) if design == "folizen" else (args.zasesun, synth.ZASESUN_SHAPES)
+    other = "llama" if design == "folizen" else "folizen_attention"
+    out = {"mode": design, "peak_kind": peak_kind, "data": "synthetic (random weights)", "models": []}
+    steps, reps = args.block_steps, args.block_reps
     sampler = ClockSampler(local_rank)
     sampler.start()
-    for name in (args.folizen.split(",") if args.folizen != "all" else ["small", "medium", "large"]):
-        c = synth.FOLIZEN_SHAPES[name]
-        n_layers = args.folizen_layers or c["layers"]
-        n_prompt, n_ctx = args.folizen_prompt, min(c["window"] + 256, 4352)
+    for name in (sizes.split(",") if sizes != "all" else ["small", "medium", "large"]):
+        c = shapes[name]
+        n_layers = args.block_layers or c["layers"]
+        n_prompt, n_ctx = args.block_prompt, args.block_ctx or min(c.get("window", 4096) + 256, 4352)
+        max_seq = n_ctx + 4 * steps + n_prompt
         toks = rng.integers(0, c["vocab"], n_prompt).astype(np.uint32)
-        arms = ["folizen", "llama"] if args.folizen_arm == "both" else [args.folizen_arm]
-        entry = {"shape": name, "layers": n_layers, **{k: c[k] for k in ("hidden", "heads", "kv_heads", "dim", "window", "ff", "vocab")}}
+        arms = [design, other] if args.block_arm == "both" else [design if args.block_arm == "design" else other]
+        entry = {"shape": name, "layers": n_layers, **{k: v for k, v in c.items() if k != "layers"}}
         for arm in arms:
-            if arm == "folizen":
-                eng = k2.Engine(ctx, synth.random_folizen(name, seed=3, max_seq=n_ctx + 4 * steps + n_prompt, layers=n_layers))
-            else:
-                lc = dict(hidden=c["hidden"], layers=n_layers, n_q=c["heads"], n_kv=c["kv_heads"], head_dim=c["dim"], inter=c["ff"], vocab=c["vocab"],
-                          max_seq=n_ctx + 4 * steps + n_prompt, eps=1e-6, theta=1e6)
+            flops = None
+            if arm == "llama":
+                lc = dict(hidden=c["hidden"], layers=n_layers, n_q=c["heads"], n_kv=c["kv_heads"], head_dim=c["dim"], inter=c["ff"], vocab=c["vocab"], max_seq=max_seq,
+                          eps=1e-6, theta=1e6)
                 eng = k2.Engine(ctx, synth.random_model(lc, "nf4g128", seed=5, untied=True, share_layers=True))
+                wb, sb = eng.weight_bytes, eng.kv_bytes_per_pos * n_ctx
+            elif arm == "folizen":
+                eng = k2.Engine(ctx, synth.random_folizen(name, seed=3, max_seq=max_seq, layers=n_layers))
+                wb, sb = _folizen_bytes(c, n_layers, n_ctx)
+                flops = _folizen_flops(c, n_layers)
+            elif arm == "folizen_attention":
+                like = synth.zasesun_like(name)
+                eng = k2.Engine(ctx, synth.random_folizen(like, seed=3, max_seq=max_seq, layers=n_layers))
+                wb, sb = _attention_like_bytes(like, n_layers, n_ctx)
+                flops = _product_flops(wb, like)
+            else:
+                eng = k2.Engine(ctx, synth.random_zasesun(name, seed=3, max_seq=max_seq, layers=n_layers))
+                wb, sb = _zasesun_bytes(c, n_layers, n_ctx)
+                flops = _product_flops(wb, c)
             eng.forward_token_ids(toks)                                   # warm-up: kernels loaded
             l0 = ctx.launch_count
-            ms_p = timed(lambda: eng.forward_token_ids(toks), args.folizen_reps)
-            launches_prompt = (ctx.launch_count - l0) // args.folizen_reps
+            ms_p = timed(lambda: eng.forward_token_ids(toks), reps)
+            launches_prompt = (ctx.launch_count - l0) // reps
             pos = 0
             while pos < n_ctx:
                 n = min(n_ctx - pos, n_prompt)
@@ -998,24 +1034,20 @@ def run_folizen(args, local_rank):
             eng.decode_greedy(1, pos, 3)
             pos += 3
             best = None
-            for _ in range(args.folizen_reps):
+            for _ in range(reps):
                 ms = timed(lambda: eng.decode_greedy(1, pos, steps), 1)
                 pos += steps
                 best = ms if best is None else min(best, ms)
             tok_s = steps / (best / 1e3)
             res = {"prompt_tokens": n_prompt, "prompt_tok_s": round(n_prompt / (ms_p / 1e3)), "prompt_launches": int(launches_prompt), "decode_ctx": n_ctx,
-                   "decode_tok_s": round(tok_s, 1), "ms_per_token": round(best / steps, 4)}
-            if arm == "folizen":
-                wb, sb = _folizen_bytes(c, n_layers, n_ctx)
-                fl = _folizen_flops(c, n_layers)
-                res.update(bytes_per_token=wb + sb, decode_frac_of_copy_peak=round((wb + sb) * tok_s / 1e9 / peak, 4),
-                           prompt_tflops=round(fl * n_prompt / ms_p / 1e9, 1), prompt_frac_of_bf16_sustained=round(fl * n_prompt / ms_p / 1e9 / tf_peak, 4))
-            else:
-                per = eng.weight_bytes + eng.kv_bytes_per_pos * n_ctx
+                   "decode_tok_s": round(tok_s, 1), "ms_per_token": round(best / steps, 4), "bytes_per_token": wb + sb,
+                   "decode_frac_of_copy_peak": round((wb + sb) * tok_s / 1e9 / peak, 4)}
+            if flops is None:
                 ops = _matmul_ops_per_token(dict(lc))
-                res.update(bytes_per_token=per, decode_frac_of_copy_peak=round(per * tok_s / 1e9 / peak, 4), prompt_int8_TOPs=round(ops * n_prompt / ms_p / 1e9, 1),
-                           prompt_frac_of_nominal_int8=round(ops * n_prompt / ms_p / 1e9 / 4500.0, 4))
-            if args.folizen_table:
+                res.update(prompt_int8_TOPs=round(ops * n_prompt / ms_p / 1e9, 1), prompt_frac_of_nominal_int8=round(ops * n_prompt / ms_p / 1e9 / 4500.0, 4))
+            else:
+                res.update(prompt_tflops=round(flops * n_prompt / ms_p / 1e9, 1), prompt_frac_of_bf16_sustained=round(flops * n_prompt / ms_p / 1e9 / tf_peak, 4))
+            if args.block_table:
                 res["step_table"] = eng.profile_step(1, pos, 8).splitlines()
             entry[arm] = res
             eng.close()
@@ -1097,12 +1129,14 @@ def main():
     ap.add_argument("--kv-bits", type=int, default=8, choices=[4, 8], help="--decode-only: KV cache format")
     ap.add_argument("--split-kv", action="store_true", help="--decode-only: split-KV attention beyond 512 positions (the engine's opt-in flag)")
     ap.add_argument("--folizen", default=None, metavar="SIZES", help="block models: small,medium,large or all - prompt and decode throughput beside a Llama shape of equal size")
-    ap.add_argument("--folizen-arm", default="both", choices=["both", "folizen", "llama"])
-    ap.add_argument("--folizen-layers", type=int, default=0, help="fewer layers than the shape's (profiling)")
-    ap.add_argument("--folizen-prompt", type=int, default=2048)
-    ap.add_argument("--folizen-steps", type=int, default=64)
-    ap.add_argument("--folizen-reps", type=int, default=3)
-    ap.add_argument("--folizen-table", action="store_true", help="add the per-kernel table of one decode step")
+    ap.add_argument("--zasesun", default=None, metavar="SIZES", help="the same for latent attention and experts, beside a Folizen shape of equal size")
+    ap.add_argument("--block-arm", default="both", choices=["both", "design", "other"], help="--folizen / --zasesun: which of the two models")
+    ap.add_argument("--block-layers", type=int, default=0, help="fewer layers than the shape's (profiling)")
+    ap.add_argument("--block-prompt", type=int, default=2048)
+    ap.add_argument("--block-ctx", type=int, default=0, help="position of the first timed decode step (default: one window + 256)")
+    ap.add_argument("--block-steps", type=int, default=64)
+    ap.add_argument("--block-reps", type=int, default=3)
+    ap.add_argument("--block-table", action="store_true", help="add the per-kernel table of one decode step")
     ap.add_argument("--case", default=None, help="profile one case, e.g. b4:2048x49152 (fmt:KxN)")
     ap.add_argument("--tokens", type=int, default=1, help="tokens per launch in --case mode (1..4)")
     ap.add_argument("--no-graph", action="store_true", help="--case mode: skip the CUDA-graph replay timing")
@@ -1112,8 +1146,8 @@ def main():
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
     if args.decode_only or args.prefill_only:
         run_decode_only(args, local_rank)
-    elif args.folizen:
-        run_folizen(args, local_rank)
+    elif args.folizen or args.zasesun:
+        run_block_models(args, local_rank, "folizen" if args.folizen else "zasesun")
     elif args.case:
         run_case(args, local_rank)
     elif args.impl == "reference":

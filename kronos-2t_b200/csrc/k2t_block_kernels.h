@@ -123,7 +123,7 @@ struct LatentAttnArgs {
     Act q_lat;                         // activation of the query product [n_tok][q_rank]
     Act q_rows;                        // few tokens: [n_tok * heads][row];  prompts: [n_tok][heads * (head_cols(dim) + head_cols(rot_dim))]
     Act kv;                            // prompts: expanded keys, then values, of all positions seen
-    float *part_o, *part_m, *part_l;   // few tokens: [n_tok * heads][splits][kv_rank], [..][splits]
+    float *part_o, *part_m, *part_l;   // few tokens: [n_tok * heads][splits][kv_rank rounded up to four], [..][splits]
     Act out;                           // [n_tok][heads * vdim]
     uint32_t *err_flag;
 };
@@ -150,6 +150,7 @@ cudaError_t launch_route(cudaStream_t s, bool f32, const RouteArgs &a, uint32_t 
 constexpr uint32_t ROUTE_MAX_EXPERTS = 1024;
 // packed rows of a batch: (token, k) pairs sorted by expert, every expert's stretch starting at a multiple of eight
 uint32_t expert_rows(uint32_t n_tok, uint32_t top, uint32_t experts);
+uint32_t expert_tile(uint32_t n_tok, uint32_t top, uint32_t experts);          // rows per item: most experts' shares in few items
 uint32_t expert_items(uint32_t n_tok, uint32_t top, uint32_t experts);
 cudaError_t launch_expert_plan(cudaStream_t s, const RouteArgs &a, uint32_t n_tok, ExpertItem *items, uint32_t *n_items, bool pdl);
 cudaError_t launch_expert_gather(cudaStream_t s, const RouteArgs &a, const Act &x, uint32_t cols, const Act &out, uint32_t n_tok, bool pdl);

@@ -192,14 +192,14 @@ bool feed_experts(KronosCudaEngine *e, Block &B, const Act &ax, uint32_t T, cons
                engine_count(e, launch_expert_down(s, b.f32, r, ed, ae, B.shared_down ? dense_view(B.shared_down->dm) : DenseView{}, b.proj, b.hs, T, e->ctx->sm_count, e->pdl), "experts down") &&
                norm_add(e, post, pre, ax, T);
     }
-    const uint32_t packed = expert_rows(T, B.top, B.experts), items = expert_items(T, B.top, B.experts);
+    const uint32_t packed = expert_rows(T, B.top, B.experts), items = expert_items(T, B.top, B.experts), tile = expert_tile(T, B.top, B.experts);
     const Act ap = act_of(b, b.act_p, packed, h), ae = act_of(b, b.act_e, packed, B.ff);
     NormArgs n = norm_args(e, post, pre, ax);
     n.top = B.top; n.pairs = b.pairs; n.pair_stride = b.hs; n.row = b.route_row; n.weight = b.route_w;
     return engine_count(e, launch_expert_plan(s, r, T, b.items, b.n_items, e->pdl), "expert plan") &&
            engine_count(e, launch_expert_gather(s, r, ax, h, ap, T, e->pdl), "expert gather") &&
-           engine_count(e, launch_dense_experts(s, eu, ap, b.items, b.n_items, items, DenseOut{r.act, nullptr, 0, 0.0f, ae}, e->ctx->d_err, e->pdl), "experts up") &&
-           engine_count(e, launch_dense_experts(s, ed, ae, b.items, b.n_items, items, dense_rows(b.pairs, b.hs), e->ctx->d_err, e->pdl), "experts down") &&
+           engine_count(e, launch_dense_experts(s, eu, ap, b.items, b.n_items, items, tile, DenseOut{r.act, nullptr, 0, 0.0f, ae}, e->ctx->d_err, e->pdl), "experts up") &&
+           engine_count(e, launch_dense_experts(s, ed, ae, b.items, b.n_items, items, tile, dense_rows(b.pairs, b.hs), e->ctx->d_err, e->pdl), "experts down") &&
            (B.shared_down ? product(e, B.shared_down, r.shared, T, b.proj, b.hs, "shared expert down")
                           : cuda_ok(e->ctx, cudaMemsetAsync(b.proj, 0, (size_t)T * b.hs * 4, s), "clear")) &&
            engine_count(e, launch_block_norm(s, false, n, T, e->pdl), "residual norm");
@@ -535,7 +535,7 @@ extern "C" KronosCudaEngine *kronos_cuda_engine_create_blocks(KronosCudaContext 
             s_cols = std::max(s_cols, d.q_rank);
             qa_bytes = std::max(qa_bytes, act_bytes(b->f32, std::min(LATENT_TOKENS, MB) * B.heads, lat.row));
             part_rows = std::max(part_rows, std::max((size_t)32 * ctx->sm_count, (size_t)LATENT_TOKENS * B.heads));
-            part_floats = std::max(part_floats, part_rows * d.kv_rank);
+            part_floats = std::max(part_floats, part_rows * ((d.kv_rank + 3u) & ~3u));
             if (B.flash) {
                 qa_bytes = std::max(qa_bytes, act_bytes(false, MB, B.heads * (dc + latent_head_cols(d.rot_dim))));
                 kv_bytes = std::max(kv_bytes, act_bytes(false, B.ring.ring_len, kv.rows));
@@ -563,7 +563,7 @@ extern "C" KronosCudaEngine *kronos_cuda_engine_create_blocks(KronosCudaContext 
                 s_cols = std::max(s_cols, B.shared_ff);
                 routes = std::max(routes, MB * B.top);
                 packed_max = std::max(packed_max, expert_rows(MB, B.top, B.experts));
-                items_max = std::max(items_max, expert_items(MB, B.top, B.experts));
+                items_max = std::max(items_max, MB * B.top / EXPERT_TILE_MIN + B.experts);
                 expert_ff = std::max(expert_ff, B.ff);
             }
         }

@@ -435,14 +435,16 @@ cudaError_t launch_dense_out(cudaStream_t s, const DeviceMatrix &dm, const Act &
     return cudaSuccess;
 }
 
-cudaError_t launch_dense_experts(cudaStream_t s, const ExpertView &m, const Act &x, const ExpertItem *items, const uint32_t *n_items, uint32_t max_items,
-                                 const DenseOut &out, uint32_t *err_flag, bool pdl) {
-    if (max_items == 0 || max_items > 65535u) return cudaErrorInvalidValue;
-    constexpr int NT = (int)EXPERT_TILE;
-    const GemmArgs a{nullptr, static_cast<const uint8_t *>(x.p), m.rows, m.rows_pad, m.panels, x.ld, 0u, out, err_flag, m.base, items, n_items};
+template <int NT> static cudaError_t gemm_experts_nt(cudaStream_t s, const GemmArgs &a, uint32_t max_items, bool pdl) {
     cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(dense_gemm_kernel<NT, true>), gm_smem<NT>());
     if (e != cudaSuccess) return e;
-    return launch_kernel(dense_gemm_kernel<NT, true>, dim3(m.rows_pad / DENSE_ROW_TILE, max_items), dim3(GM_THREADS), gm_smem<NT>(), s, pdl, a);
+    return launch_kernel(dense_gemm_kernel<NT, true>, dim3(a.rows_pad / DENSE_ROW_TILE, max_items), dim3(GM_THREADS), gm_smem<NT>(), s, pdl, a);
+}
+cudaError_t launch_dense_experts(cudaStream_t s, const ExpertView &m, const Act &x, const ExpertItem *items, const uint32_t *n_items, uint32_t max_items,
+                                 uint32_t tile, const DenseOut &out, uint32_t *err_flag, bool pdl) {
+    if (max_items == 0 || max_items > 65535u) return cudaErrorInvalidValue;
+    const GemmArgs a{nullptr, static_cast<const uint8_t *>(x.p), m.rows, m.rows_pad, m.panels, x.ld, 0u, out, err_flag, m.base, items, n_items};
+    return tile == 64 ? gemm_experts_nt<64>(s, a, max_items, pdl) : tile == 128 ? gemm_experts_nt<128>(s, a, max_items, pdl) : cudaErrorInvalidValue;
 }
 
 }  // namespace k2t

@@ -79,10 +79,10 @@ struct ExpertView {
 };
 // A stretch of rows [row0, row_end) of a packed activation that one expert works on; row0 is a multiple of eight.
 struct ExpertItem { uint32_t expert, row0, row_end, pad; };
-constexpr uint32_t EXPERT_TILE = 64;        // rows of the packed activation per item
-// tensor-core product of every item's rows with its expert; items and their number live on the device (at most max_items).
+constexpr uint32_t EXPERT_TILE_MIN = 64;    // rows of the packed activation per item: 64 or 128
+// tensor-core product of every item's rows (at most `tile`) with its expert; items and their number live on the device (at most max_items).
 // Row p of the packed activation gives row p of the output.
 cudaError_t launch_dense_experts(cudaStream_t s, const ExpertView &m, const Act &x, const ExpertItem *items, const uint32_t *n_items, uint32_t max_items,
-                                 const DenseOut &out, uint32_t *err_flag, bool pdl);
+                                 uint32_t tile, const DenseOut &out, uint32_t *err_flag, bool pdl);
 
 }  // namespace k2t

@@ -14,10 +14,10 @@
 namespace k2t {
 namespace {
 
-constexpr uint32_t EX_THREADS = 256, EX_PF = 4, EX_MAX_SLOTS = 33;      // top <= 32, and the shared expert
+constexpr uint32_t RT_THREADS = 1024, EX_THREADS = 256, EX_PF = 8, EX_MAX_SLOTS = 33;      // top <= 32, and the shared expert
 
 template <bool F32>
-__global__ void __launch_bounds__(EX_THREADS) route_kernel(const RouteArgs a) {
+__global__ void __launch_bounds__(RT_THREADS) route_kernel(const RouteArgs a) {
     __shared__ float s[ROUTE_MAX_EXPERTS];
     const uint32_t t = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
     pdl_wait();
@@ -47,7 +47,7 @@ __global__ void __launch_bounds__(EX_THREADS) route_kernel(const RouteArgs a) {
         }
     } else {
         const float *h = z + a.experts;
-        for (uint32_t i = tid - 32; i < a.shared_ff; i += EX_THREADS - 32)
+        for (uint32_t i = tid - 32; i < a.shared_ff; i += blockDim.x - 32)
             act_store<F32>(a.shared, t, i, a.act == Epi::GeluGated ? gelu_tanh(__ldcg(h + 2 * i)) * __ldcg(h + 2 * i + 1) : relu_squared(__ldcg(h + i)));
     }
 }
@@ -67,7 +67,7 @@ __device__ __forceinline__ uint32_t block_scan_1024(uint32_t v, uint32_t *s_warp
 }
 
 // One CTA of 32 warps, warp = a stretch of the pairs; thread = expert in between.
-__global__ void __launch_bounds__(1024) expert_plan_kernel(const RouteArgs a, uint32_t pairs, ExpertItem *__restrict__ items, uint32_t *__restrict__ n_items) {
+__global__ void __launch_bounds__(1024) expert_plan_kernel(const RouteArgs a, uint32_t pairs, uint32_t tile, ExpertItem *__restrict__ items, uint32_t *__restrict__ n_items) {
     extern __shared__ uint32_t s_hist[];          // [32][experts]
     __shared__ uint32_t s_first[ROUTE_MAX_EXPERTS], s_warp[32];
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = a.experts;
@@ -77,31 +77,39 @@ __global__ void __launch_bounds__(1024) expert_plan_kernel(const RouteArgs a, ui
     __syncthreads();
     const uint32_t per = ((pairs + 1023) / 1024) * 32, p0 = warp * per, p1 = min(pairs, p0 + per);
     uint32_t *hist = s_hist + warp * E;
-    for (uint32_t p = p0; p < p1; p += 32) {
-        const bool in = p + lane < p1;
-        const uint32_t active = __ballot_sync(0xffffffffu, in);
-        if (in) {
-            const uint32_t e = __ldcg(a.ids + p + lane), same = __match_any_sync(active, e), rank = __popc(same & ((1u << lane) - 1u));
-            const uint32_t base = hist[e];
-            __syncwarp(active);
-            if (rank == 0) hist[e] = base + __popc(same);
-            a.row[p + lane] = base + rank;
+    constexpr uint32_t AHEAD = 4;          // ids of the next steps are on their way
+    for (uint32_t p = p0; p < p1; p += 32 * AHEAD) {
+        uint32_t id[AHEAD];
+#pragma unroll
+        for (uint32_t i = 0; i < AHEAD; ++i) id[i] = p + 32 * i + lane < p1 ? __ldcg(a.ids + p + 32 * i + lane) : 0u;
+#pragma unroll
+        for (uint32_t i = 0; i < AHEAD; ++i) {
+            const uint32_t q = p + 32 * i + lane;
+            const bool in = q < p1;
+            const uint32_t active = __ballot_sync(0xffffffffu, in);
+            if (in) {
+                const uint32_t same = __match_any_sync(active, id[i]), rank = __popc(same & ((1u << lane) - 1u)), base = hist[id[i]];
+                __syncwarp(active);
+                if (rank == 0) hist[id[i]] = base + __popc(same);
+                a.row[q] = base + rank;
+            }
+            __syncwarp();
         }
-        __syncwarp();
     }
     __syncthreads();
     uint32_t count = 0;
     if (tid < E)
         for (uint32_t w = 0; w < 32; ++w) { const uint32_t c = s_hist[w * E + tid]; s_hist[w * E + tid] = count; count += c; }
     uint32_t total_rows, total_items;
-    const uint32_t first = block_scan_1024((count + 7u) & ~7u, s_warp, total_rows), n = (count + EXPERT_TILE - 1) / EXPERT_TILE;
+    const uint32_t first = block_scan_1024((count + 7u) & ~7u, s_warp, total_rows), n = (count + tile - 1) / tile;
     const uint32_t at = block_scan_1024(n, s_warp, total_items);
     if (tid < E) {
         s_first[tid] = first;
-        for (uint32_t i = 0; i < n; ++i) items[at + i] = ExpertItem{tid, first + i * EXPERT_TILE, min(first + count, first + (i + 1) * EXPERT_TILE), 0u};
+        for (uint32_t i = 0; i < n; ++i) items[at + i] = ExpertItem{tid, first + i * tile, min(first + count, first + (i + 1) * tile), 0u};
     }
     if (tid == 0) *n_items = total_items;
     __syncthreads();
+#pragma unroll 4
     for (uint32_t p = p0 + lane; p < p1; p += 32) {
         const uint32_t e = __ldcg(a.ids + p);
         a.row[p] += s_first[e] + hist[e];
@@ -132,7 +140,7 @@ struct ExpertGemvArgs {
 
 // UP: blockIdx.y = choice k of token blockIdx.z.  DOWN: all choices of token blockIdx.z, their panels one after the other.
 template <bool DOWN>
-__global__ void __launch_bounds__(EX_THREADS, 4) expert_gemv_kernel(const ExpertGemvArgs a) {
+__global__ void __launch_bounds__(EX_THREADS, 2) expert_gemv_kernel(const ExpertGemvArgs a) {
     __shared__ float s_part[8][8], s_w[EX_MAX_SLOTS];
     __shared__ const uint4 *s_base[EX_MAX_SLOTS];
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wk = 1u << a.wk_log2, c = lane & 7u, r = lane >> 3, t = blockIdx.z, top = a.route.top;
@@ -238,24 +246,29 @@ __global__ void __launch_bounds__(EX_THREADS) expert_gemv_f32_kernel(const Exper
 // warps per row group: about one wave of CTAs, but a handful of panels per warp at least
 uint32_t split_warps(uint32_t groups, uint32_t panels, int sm_count) {
     uint32_t wl = 0;
-    while (wl < 3 && (2u << wl) * EX_PF <= panels && groups << wl <= 8u * (uint32_t)sm_count) ++wl;
+    while (wl < 3 && (2u << wl) * 4 <= panels && groups << wl <= 8u * (uint32_t)sm_count) ++wl;
     return wl;
 }
 
 }  // namespace
 
 cudaError_t launch_route(cudaStream_t s, bool f32, const RouteArgs &a, uint32_t n_tok, bool pdl) {
-    return launch_kernel(f32 ? route_kernel<true> : route_kernel<false>, dim3(n_tok), dim3(EX_THREADS), 0, s, pdl, a);
+    const uint32_t threads = n_tok > 64 ? 256u : std::min(RT_THREADS, 64u + ((a.shared_ff + 31u) & ~31u));
+    return launch_kernel(f32 ? route_kernel<true> : route_kernel<false>, dim3(n_tok), dim3(threads), 0, s, pdl, a);
 }
 
 uint32_t expert_rows(uint32_t n_tok, uint32_t top, uint32_t experts) { return (n_tok * top + 7 * std::min(experts, n_tok * top) + 7u) & ~7u; }
-uint32_t expert_items(uint32_t n_tok, uint32_t top, uint32_t experts) { return n_tok * top / EXPERT_TILE + std::min(experts, n_tok * top); }
+uint32_t expert_tile(uint32_t n_tok, uint32_t top, uint32_t experts) {
+    const uint32_t share = n_tok * top / experts;
+    return share >= 96 ? 128u : EXPERT_TILE_MIN;
+}
+uint32_t expert_items(uint32_t n_tok, uint32_t top, uint32_t experts) { return n_tok * top / expert_tile(n_tok, top, experts) + std::min(experts, n_tok * top); }
 
 cudaError_t launch_expert_plan(cudaStream_t s, const RouteArgs &a, uint32_t n_tok, ExpertItem *items, uint32_t *n_items, bool pdl) {
     const size_t smem = (size_t)32 * a.experts * 4;
     cudaError_t e = allow_dynamic_smem(reinterpret_cast<const void *>(expert_plan_kernel), smem);
     if (e != cudaSuccess) return e;
-    return launch_kernel(expert_plan_kernel, dim3(1), dim3(1024), smem, s, pdl, a, n_tok * a.top, items, n_items);
+    return launch_kernel(expert_plan_kernel, dim3(1), dim3(1024), smem, s, pdl, a, n_tok * a.top, expert_tile(n_tok, a.top, a.experts), items, n_items);
 }
 
 cudaError_t launch_expert_gather(cudaStream_t s, const RouteArgs &a, const Act &x, uint32_t cols, const Act &out, uint32_t n_tok, bool pdl) {

@@ -23,25 +23,33 @@ __device__ __forceinline__ float exp2_approx(float x) { float y; asm("ex2.approx
 
 // ------------------------------------------------------------------------------------------------ latents, cache row
 // grid (token, 2): the query latent; the cache row
+constexpr uint32_t PREP_THREADS = 512;
 template <bool F32>
-__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentAttnArgs a) {
+__global__ void __launch_bounds__(PREP_THREADS) latent_prep_kernel(const LatentAttnArgs a) {
     __shared__ float scratch[32];
     const LatentShape &d = a.d;
-    const uint32_t t = blockIdx.x, tid = threadIdx.x, n = blockIdx.y == 0 ? d.q_rank : d.kv_rank;
+    const uint32_t t = blockIdx.x, tid = threadIdx.x, step = blockDim.x, n = blockIdx.y == 0 ? d.q_rank : d.kv_rank;
     const float *w = blockIdx.y == 0 ? a.q_norm : a.kv_norm;
     pdl_wait();
     pdl_trigger();
     const float *x = a.in + t * a.in_stride + (blockIdx.y == 0 ? 0 : d.q_rank);
     const uint32_t pos = __ldcg(a.pos) + t;
-    float ss[1] = {0.0f};
-    for (uint32_t k = tid; k < n; k += 256) { const float v = __ldcg(x + k); ss[0] = __fmaf_rn(v, v, ss[0]); }
+    constexpr uint32_t KEEP = 4;               // the thread's first values stay in registers
+    float keep[KEEP], ss[1] = {0.0f};
+#pragma unroll
+    for (uint32_t i = 0; i < KEEP; ++i) { const uint32_t k = tid + i * step; keep[i] = k < n ? __ldcg(x + k) : 0.0f; }
+#pragma unroll
+    for (uint32_t i = 0; i < KEEP; ++i) ss[0] = __fmaf_rn(keep[i], keep[i], ss[0]);
+    for (uint32_t k = tid + KEEP * step; k < n; k += step) { const float v = __ldcg(x + k); ss[0] = __fmaf_rn(v, v, ss[0]); }
     block_sum<1>(ss, scratch);
     const float inv = 1.0f / sqrtf(ss[0] / (float)n + a.eps);
     const Act &out = blockIdx.y == 0 ? a.q_lat : a.cache;
     const uint32_t row = blockIdx.y == 0 ? t : pos;
-    for (uint32_t k = tid; k < n; k += 256) act_store<F32>(out, row, k, __ldcg(x + k) * inv * __ldg(w + k));
+#pragma unroll
+    for (uint32_t i = 0; i < KEEP; ++i) { const uint32_t k = tid + i * step; if (k < n) act_store<F32>(out, row, k, keep[i] * inv * __ldg(w + k)); }
+    for (uint32_t k = tid + KEEP * step; k < n; k += step) act_store<F32>(out, row, k, __ldcg(x + k) * inv * __ldg(w + k));
     if (blockIdx.y == 1)
-        for (uint32_t i = tid; i < d.rot_dim / 2; i += 256) {
+        for (uint32_t i = tid; i < d.rot_dim / 2; i += step) {
             const float u = __ldcg(x + d.kv_rank + 2 * i), v = __ldcg(x + d.kv_rank + 2 * i + 1);
             const float c = __ldg(a.rot + (size_t)pos * d.rot_dim + 2 * i), s = __ldg(a.rot + (size_t)pos * d.rot_dim + 2 * i + 1);
             act_store<F32>(a.cache, pos, d.rot_at + 2 * i, u * c - v * s);
@@ -156,6 +164,7 @@ struct SplitParams {
     LatentAttnArgs a;
     uint32_t t0, rows, splits, stages;      // rows = tokens * heads
 };
+__host__ __device__ inline uint32_t part_stride(const LatentShape &d) { return (d.kv_rank + 3u) & ~3u; }
 // tiles [first, last) of this split, of the tiles the launch's last token sees (alike for all rows: the merge counts on it)
 __device__ __forceinline__ void split_range(uint32_t seen, uint32_t split, uint32_t splits, uint32_t &first, uint32_t &last) {
     const uint32_t tiles = (seen + SP_N - 1) / SP_N, per = (tiles + splits - 1) / splits;
@@ -330,7 +339,7 @@ __global__ void __launch_bounds__(SP_THREADS) latent_split_kernel(const SplitPar
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
                 const uint32_t row = b * 16 + (lane >> 2) + ((e >> 1) & 1) * 8, k = (warp + 8 * u) * 16 + (e >> 2) * 8 + (lane & 3u) * 2 + (e & 1);
-                if (row < n_row && k < d.kv_rank) a.part_o[((size_t)(r0 + row) * p.splits + split) * d.kv_rank + k] = o[b][u][e >> 2][e & 3];
+                if (row < n_row && k < d.kv_rank) a.part_o[((size_t)(r0 + row) * p.splits + split) * part_stride(d) + k] = o[b][u][e >> 2][e & 3];
             }
 }
 
@@ -380,48 +389,89 @@ __global__ void __launch_bounds__(256) latent_split_f32_kernel(const SplitParams
         }
         __syncthreads();
     }
-    for (uint32_t k = tid; k < d.kv_rank; k += 256) a.part_o[((size_t)row * p.splits + split) * d.kv_rank + k] = s_o[k];
+    for (uint32_t k = tid; k < d.kv_rank; k += 256) a.part_o[((size_t)row * p.splits + split) * part_stride(d) + k] = s_o[k];
     if (tid == 0) { a.part_m[(size_t)row * p.splits + split] = m; a.part_l[(size_t)row * p.splits + split] = l; }
 }
 
-// grid (32 value rows, head, token): merge of the splits, then W_uv of the head
+// grid (64 value rows, head, token): merge of the splits, then W_uv of the head.  Thread = (four columns, group of splits); the
+// first partial results are requested before their factors are known, the weights before the dependency wait.
+constexpr uint32_t VL_THREADS = 512, VL_PF = 8;
 template <bool F32>
-__global__ void __launch_bounds__(256) latent_value_kernel(const SplitParams p) {
+__global__ void __launch_bounds__(VL_THREADS) latent_value_kernel(const SplitParams p) {
     extern __shared__ __align__(16) float sf[];
     const LatentAttnArgs &a = p.a;
     const LatentShape &d = a.d;
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, t = blockIdx.z, row = t * d.heads + h;
-    const uint32_t padded = (d.kv_rank + PANEL - 1) / PANEL * PANEL;
+    const uint32_t panels = (d.kv_rank + PANEL - 1) / PANEL, padded = panels * PANEL, quads = part_stride(d) / 4;
     float *s_c = sf, *s_f = s_c + padded;
-    for (uint32_t k = tid; k < padded; k += 256) s_c[k] = 0.0f;
-    const uint32_t sub = lane & 7u, v = blockIdx.x * 32 + warp * 4 + (lane >> 3), vv = min(v, d.vdim - 1);
+    float4 *s_part = reinterpret_cast<float4 *>(s_f + ((p.splits + 4) & ~3u));          // [VL_THREADS]
+    for (uint32_t k = tid; k < padded; k += VL_THREADS) s_c[k] = 0.0f;
+    const uint32_t sub = lane & 7u, v = blockIdx.x * 64 + warp * 4 + (lane >> 3), vv = min(v, d.vdim - 1);
     const uint32_t w_row = d.heads * latent_head_cols(d.dim) + h * latent_head_cols(d.vdim) + vv;
+    const uint4 *wp = static_cast<const uint4 *>(a.kv_up.base) + (size_t)w_row * 8 + (sub ^ (w_row & 7u));
+    uint4 w[VL_PF];
+    if (!F32)
+#pragma unroll
+        for (uint32_t i = 0; i < VL_PF; ++i) w[i] = i < panels ? ldg_stream(wp + (size_t)i * a.kv_up.rows_pad * 8) : make_uint4(0, 0, 0, 0);
     pdl_wait();
     pdl_trigger();
+    uint32_t first, last;                    // splits that hold a position at all
+    const uint32_t seen = __ldcg(a.pos) + p.t0 + p.rows / d.heads;
+    split_range(seen, 0, p.splits, first, last);
+    const uint32_t used = min(p.splits, ((seen + SP_N - 1) / SP_N + last - 1) / max(1u, last));
     const float *pm = a.part_m + (size_t)row * p.splits, *pl = a.part_l + (size_t)row * p.splits;
-    if (warp == 0) {
+    const float4 *po = reinterpret_cast<const float4 *>(a.part_o) + (size_t)row * p.splits * quads;
+    // quads q0, q0 + cols, ..: `cols` threads side by side, `groups` of them over the splits
+    const uint32_t cols = min(quads, VL_THREADS), groups = VL_THREADS / cols, g = tid / cols, q0 = tid % cols;
+    constexpr uint32_t PRE = 4;
+    float4 pre[PRE];
+#pragma unroll
+    for (uint32_t i = 0; i < PRE; ++i) pre[i] = g < groups && g + i * groups < used ? __ldcg(po + (size_t)(g + i * groups) * quads + q0) : make_float4(0, 0, 0, 0);
+    if (warp == VL_THREADS / 32 - 1) {
         float m = -INFINITY, l = 0.0f;
-        for (uint32_t s = lane; s < p.splits; s += 32) m = fmaxf(m, __ldcg(pm + s));
+        for (uint32_t s = lane; s < used; s += 32) m = fmaxf(m, __ldcg(pm + s));
 #pragma unroll
         for (int k = 16; k > 0; k >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, k));
-        for (uint32_t s = lane; s < p.splits; s += 32) { const float f = F32 ? expf(__ldcg(pm + s) - m) : exp2f(__ldcg(pm + s) - m); s_f[s] = f; l = __fmaf_rn(f, __ldcg(pl + s), l); }
+        for (uint32_t s = lane; s < used; s += 32) { const float f = F32 ? expf(__ldcg(pm + s) - m) : exp2f(__ldcg(pm + s) - m); s_f[s] = f; l = __fmaf_rn(f, __ldcg(pl + s), l); }
         l = warp_sum(l);
         if (lane == 0) s_f[p.splits] = 1.0f / l;
     }
     __syncthreads();
     const float inv = s_f[p.splits];
-    uint32_t first, last;                    // splits that hold a position at all
-    const uint32_t seen = __ldcg(a.pos) + p.t0 + p.rows / d.heads;
-    split_range(seen, 0, p.splits, first, last);
-    const uint32_t used = min(p.splits, ((seen + SP_N - 1) / SP_N + last - 1) / max(1u, last));
-    for (uint32_t k = tid; k < d.kv_rank; k += 256) {
-        float o = 0.0f;
+    for (uint32_t qb = 0; qb < quads; qb += cols) {
+        const uint32_t q = qb + q0;
+        float4 o = make_float4(0, 0, 0, 0);
+        auto add = [&](float f, const float4 &x) { o.x = __fmaf_rn(f, x.x, o.x); o.y = __fmaf_rn(f, x.y, o.y); o.z = __fmaf_rn(f, x.z, o.z); o.w = __fmaf_rn(f, x.w, o.w); };
+        if (g < groups && q < quads) {
+            uint32_t s = g;
+            if (qb == 0) {
+#pragma unroll
+                for (uint32_t i = 0; i < PRE; ++i, s += groups)
+                    if (s < used) add(s_f[s], pre[i]);
+            }
 #pragma unroll 8
-        for (uint32_t s = 0; s < used; ++s) o = __fmaf_rn(s_f[s], __ldcg(a.part_o + ((size_t)row * p.splits + s) * d.kv_rank + k), o);
-        s_c[k] = o * inv;
+            for (; s < used; s += groups) add(s_f[s], __ldcg(po + (size_t)s * quads + q));
+        }
+        s_part[tid] = o;
+        __syncthreads();
+        if (tid < cols && q < quads) {
+            for (uint32_t i = 1; i < groups; ++i) { const float4 x = s_part[i * cols + tid]; o.x += x.x; o.y += x.y; o.z += x.z; o.w += x.w; }
+            const float e[4] = {o.x, o.y, o.z, o.w};
+            for (uint32_t i = 0; i < 4 && q * 4 + i < d.kv_rank; ++i) s_c[q * 4 + i] = e[i] * inv;
+        }
+        __syncthreads();
     }
-    __syncthreads();
-    const float s = row_dot8<F32>(a.kv_up, w_row, 0, (d.kv_rank + PANEL - 1) / PANEL, s_c, sub);
+    float s = 0.0f;
+    if (F32) {
+        s = row_dot8<true>(a.kv_up, w_row, 0, panels, s_c, sub);
+    } else {
+#pragma unroll
+        for (uint32_t i = 0; i < VL_PF; ++i)
+            if (i < panels) s = dot8(w[i], s_c + i * PANEL + sub * 8, s);
+        for (uint32_t i = VL_PF; i < panels; ++i) s = dot8(ldg_stream(wp + (size_t)i * a.kv_up.rows_pad * 8), s_c + i * PANEL + sub * 8, s);
+#pragma unroll
+        for (int m = 1; m < 8; m <<= 1) s = __fadd_rn(s, __shfl_xor_sync(0xffffffffu, s, m));
+    }
     if (v < d.vdim && sub == 0) act_store<F32>(a.out, p.t0 + t, h * d.vdim + v, s);
 }
 
@@ -770,7 +820,8 @@ bool latent_attn_fits(bool f32, const LatentShape &d) {
 bool latent_flash_fits(const LatentShape &d) { const FlashShape f = flash_shape(d); return f.smem <= 226 * 1024 && f.vn <= 256 && f.tmem <= 512; }
 
 cudaError_t launch_latent_prep(cudaStream_t s, bool f32, const LatentAttnArgs &a, uint32_t n_tok, bool pdl) {
-    return launch_kernel(f32 ? latent_prep_kernel<true> : latent_prep_kernel<false>, dim3(n_tok, 2), dim3(256), 0, s, pdl, a);
+    const uint32_t n = std::max(a.d.q_rank, a.d.kv_rank), threads = n_tok > 64 ? 256u : std::min(PREP_THREADS, std::max(64u, (n + 31u) & ~31u));
+    return launch_kernel(f32 ? latent_prep_kernel<true> : latent_prep_kernel<false>, dim3(n_tok, 2), dim3(threads), 0, s, pdl, a);
 }
 
 uint32_t latent_splits(const LatentShape &d, uint32_t n_tok, uint32_t max_positions, int sm_count) {
@@ -782,8 +833,8 @@ cudaError_t launch_latent_few(cudaStream_t s, bool f32, const LatentAttnArgs &a,
     const LatentShape &d = a.d;
     if (n_tok == 0 || n_tok > LATENT_TOKENS || splits == 0) return cudaErrorInvalidValue;
     SplitParams p{a, t0, n_tok * d.heads, splits, 0};
-    const dim3 value_grid((d.vdim + 31) / 32, d.heads, n_tok);
-    const size_t value_smem = ((size_t)((d.kv_rank + PANEL - 1) / PANEL) * PANEL + splits + 1) * 4;
+    const dim3 value_grid((d.vdim + 63) / 64, d.heads, n_tok);
+    const size_t value_smem = ((size_t)((d.kv_rank + PANEL - 1) / PANEL) * PANEL + ((splits + 4) & ~3u) + 4 * VL_THREADS) * 4;
     cudaError_t e;
     if (f32) {
         e = launch_kernel(latent_absorb_f32_kernel, dim3((d.row + 255) / 256, d.heads, n_tok), dim3(256), 0, s, pdl, a, t0);
@@ -793,7 +844,7 @@ cudaError_t launch_latent_few(cudaStream_t s, bool f32, const LatentAttnArgs &a,
         if (e != cudaSuccess) return e;
         e = launch_kernel(latent_split_f32_kernel, dim3(splits, p.rows), dim3(256), smem, s, pdl, p);
         if (e != cudaSuccess) return e;
-        return launch_kernel(latent_value_kernel<true>, value_grid, dim3(256), value_smem, s, pdl, p);
+        return launch_kernel(latent_value_kernel<true>, value_grid, dim3(VL_THREADS), value_smem, s, pdl, p);
     }
     const uint32_t cols = d.rot_at / PANEL + 1;
     e = n_tok == 1 ? launch_kernel(latent_absorb_kernel<1>, dim3(cols, d.heads, 1), dim3(256), 0, s, pdl, a, t0, t0 + n_tok)
@@ -803,7 +854,7 @@ cudaError_t launch_latent_few(cudaStream_t s, bool f32, const LatentAttnArgs &a,
     p.stages = sh.stages;
     e = sh.rb == 2 ? split_launch<2>(s, p, sh.smem, pdl) : sh.rb == 1 ? split_launch<1>(s, p, sh.smem, pdl) : cudaErrorInvalidValue;
     if (e != cudaSuccess) return e;
-    return launch_kernel(latent_value_kernel<false>, value_grid, dim3(256), value_smem, s, pdl, p);
+    return launch_kernel(latent_value_kernel<false>, value_grid, dim3(VL_THREADS), value_smem, s, pdl, p);
 }
 
 cudaError_t launch_latent_prompt(cudaStream_t s, const LatentAttnArgs &a, uint32_t n_tok, bool pdl) {

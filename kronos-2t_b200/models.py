@@ -207,8 +207,8 @@ def zasesun_spec(folder, config, dtype, max_seq):
                 raise ValueError(f"layer {i}: unknown feed-forward {kind!r}")
         blocks.append(b)
     embed = mat("embed")
-    return dict(cfg=dict(hidden=embed.shape[1], vocab=embed.shape[0], max_seq=max_seq, eps=config["norm"]["eps"], residual_mult=config["residual_mult"],
-                         logit_softcap=config["logit_softcap"], precision=16 if dtype == "bfloat16" else 32),
+    return dict(cfg=dict(hidden=embed.shape[1], vocab=embed.shape[0], max_seq=max_seq, eps=config["norm"]["eps"], residual_mult=config.get("residual_mult", 1.0),
+                         logit_softcap=config.get("logit_softcap") or 0.0, precision=16 if dtype == "bfloat16" else 32),
                 blocks=blocks, final_norm=t.f32("final.norm"), head=embed, embed=t.bits("embed"))
 
 

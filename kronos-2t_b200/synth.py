@@ -177,25 +177,72 @@ FOLIZEN_SHAPES = {
 }
 
 
-def random_folizen(shape, seed=0, max_seq=8192, layers=None):
-    """Engine spec of a block model with random bf16 weights: attention with feed-forward and delta-rule blocks by turns.  Blocks
-    of a kind point at the same host arrays (each still becomes its own device copy)."""
-    c = dict(FOLIZEN_SHAPES[shape] if isinstance(shape, str) else shape)
-    n = layers or c["layers"]
-    h, H, G, d, ff, side = c["hidden"], c["heads"], c["kv_heads"], c["dim"], c["ff"], c["side_dim"]
-    rng = _rng(seed)
-
+def _block_matrix(rng):
+    """mat(rows, cols): random bf16 bit patterns with magnitudes around 1 / sqrt(cols)."""
     def mat(rows, cols):
-        base = int(np.float32(cols ** -0.5).view(np.uint32) >> 16) & 0x7F80      # magnitudes around 1 / sqrt(cols)
+        base = int(np.float32(cols ** -0.5).view(np.uint32) >> 16) & 0x7F80
         blk = rng.integers(base - 0x80, base + 0x80, min(rows * cols, 1 << 22), dtype=np.uint16) | (rng.integers(0, 2, min(rows * cols, 1 << 22), dtype=np.uint16) << 15)
         return np.resize(blk, rows * cols).reshape(rows, cols)
+    return mat
 
+
+def random_folizen(shape, seed=0, max_seq=8192, layers=None):
+    """Engine spec of a block model with random bf16 weights: attention with feed-forward and delta-rule blocks by turns, or attention
+    blocks only, with feed-forward sizes by turns, where the shape has ff_turns.  Blocks of a kind point at the same host arrays
+    (each still becomes its own device copy)."""
+    c = dict(FOLIZEN_SHAPES[shape] if isinstance(shape, str) else shape)
+    n = layers or c["layers"]
+    h, H, G, d, side = c["hidden"], c["heads"], c["kv_heads"], c["dim"], c["side_dim"]
+    mat = _block_matrix(_rng(seed))
     one = lambda k: np.ones(k, np.float32)
-    tail = dict(norm1=one(h), side_norm=one(h) * 0.5, side_gate=mat(side, h), side_proj=mat(h, side))
-    attn = dict(tail, mixer=1, heads=H, kv_heads=G, dim=d, vdim=d, window=c["window"], ff=ff, q_norm=one(d), k_norm=one(d), head_scale=one(H) * d ** -0.5,
-                head_slope=(2.0 ** (-8.0 * (np.arange(H) + 1) / H)).astype(np.float32), in_proj=mat((H + 2 * G) * d, h), o_proj=mat(h, H * d), norm2=one(h),
-                act_coef=np.array([0.5, 0.3, 0.2, 0.0], np.float32), up_proj=mat(ff, h), down_proj=mat(h, ff))
-    delta = dict(tail, mixer=2, heads=H, dim=d, decay_rank=c["rank"], decay_scale=0.6065307, unit_eps=1e-6, decay_bias=-2.0 * one(H * d), rate_bias=-1.0 * one(H * d),
-                 out_norm=one(H * d), in_proj=mat(5 * H * d + c["rank"], h), decay_proj=mat(H * d, c["rank"]), o_proj=mat(h, H * d))
-    return dict(cfg=dict(hidden=h, vocab=c["vocab"], max_seq=max_seq, eps=1e-6, side_dim=side, precision=16), blocks=[attn if i % 2 == 0 else delta for i in range(n)],
-                final_norm=one(h), head=mat(c["vocab"], h), embed=mat(c["vocab"], h), side_embed=mat(c["vocab"], side * n))
+    tail = dict(norm1=one(h))
+    if side:
+        tail.update(side_norm=one(h) * 0.5, side_gate=mat(side, h), side_proj=mat(h, side))
+
+    def attention(ff):
+        return dict(tail, mixer=1, heads=H, kv_heads=G, dim=d, vdim=d, window=c["window"], ff=ff, q_norm=one(d), k_norm=one(d), head_scale=one(H) * d ** -0.5,
+                    head_slope=(2.0 ** (-8.0 * (np.arange(H) + 1) / H)).astype(np.float32), in_proj=mat((H + 2 * G) * d, h), o_proj=mat(h, H * d), norm2=one(h),
+                    act_coef=np.array([0.5, 0.3, 0.2, 0.0], np.float32), up_proj=mat(ff, h), down_proj=mat(h, ff))
+
+    if "ff_turns" in c:
+        turns = [attention(ff) for ff in c["ff_turns"]]
+    else:
+        turns = [attention(c["ff"]), dict(tail, mixer=2, heads=H, dim=d, decay_rank=c["rank"], decay_scale=0.6065307, unit_eps=1e-6, decay_bias=-2.0 * one(H * d),
+                                          rate_bias=-1.0 * one(H * d), out_norm=one(H * d), in_proj=mat(5 * H * d + c["rank"], h), decay_proj=mat(H * d, c["rank"]),
+                                          o_proj=mat(h, H * d))]
+    return dict(cfg=dict(hidden=h, vocab=c["vocab"], max_seq=max_seq, eps=1e-6, side_dim=side, precision=16), blocks=[turns[i % len(turns)] for i in range(n)],
+                final_norm=one(h), head=mat(c["vocab"], h), embed=mat(c["vocab"], h), side_embed=mat(c["vocab"], side * n) if side else None)
+
+
+ZASESUN_SHAPES = {
+    "small": dict(hidden=1024, layers=12, heads=16, dim=64, rot_dim=32, vdim=64, q_rank=512, kv_rank=256, ff=4096, experts=32, top=4, expert_ff=704, shared_ff=1408, vocab=32768),
+    "medium": dict(hidden=2048, layers=24, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=1024, kv_rank=512, ff=8192, experts=64, top=6, expert_ff=1408, shared_ff=2816, vocab=49152),
+    "large": dict(hidden=4096, layers=16, heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, ff=14336, experts=32, top=4, expert_ff=2048, shared_ff=4096, vocab=131072),
+}
+
+
+def random_zasesun(shape, seed=0, max_seq=8192, layers=None):
+    """Engine spec with random bf16 weights: latent attention with a dense and an expert feed-forward by turns."""
+    from . import models
+    c = dict(ZASESUN_SHAPES[shape] if isinstance(shape, str) else shape)
+    n, h, H, d, dr, dv = layers or c["layers"], c["hidden"], c["heads"], c["dim"], c["rot_dim"], c["vdim"]
+    mat = _block_matrix(_rng(seed))
+    one = lambda k: np.ones(k, np.float32)
+    attn = dict(mixer=3, heads=H, dim=d, vdim=dv, rot_dim=dr, kv_rank=c["kv_rank"], q_rank=c["q_rank"], score_scale=(d + dr) ** -0.5,
+                rot_cos_sin=models.rotation_table(max_seq, dr, dr, 1e4, dict(factor=8.0, original=4096, fast=32.0, slow=1.0)), q_latent_norm=one(c["q_rank"]),
+                kv_latent_norm=one(c["kv_rank"]), pre_norm1=one(h), norm1=one(h), in_proj=mat(c["q_rank"] + c["kv_rank"] + dr, h), q_up=mat(H * (d + dr), c["q_rank"]),
+                kv_up=mat(H * (d + dv), c["kv_rank"]), o_proj=mat(h, H * dv), pre_norm2=one(h), norm2=one(h))
+    E, ff, sh = c["experts"], c["expert_ff"], c["shared_ff"]
+    turns = [dict(attn, act=1, ff=c["ff"], up_proj=mat(2 * c["ff"], h), down_proj=mat(h, c["ff"])),
+             dict(attn, act=2, ff=ff, experts=E, experts_top=c["top"], shared_ff=sh, up_proj=mat(E * ff, h), down_proj=mat(E * h, ff), router=mat(E + sh, h), shared_down=mat(h, sh))]
+    table = mat(c["vocab"], h)
+    return dict(cfg=dict(hidden=h, vocab=c["vocab"], max_seq=max_seq, eps=1e-6, residual_mult=0.5, logit_softcap=30.0, precision=16),
+                blocks=[turns[i % 2] for i in range(n)], final_norm=one(h), head=table, embed=table)
+
+
+def zasesun_like(shape):
+    """The Folizen shape of equal width, depth, heads and active feed-forward sizes: attention over every position, as many
+    key/value heads as give the nearest cache (one eighth of the query heads, at least one)."""
+    c = dict(ZASESUN_SHAPES[shape] if isinstance(shape, str) else shape)
+    return dict(hidden=c["hidden"], layers=c["layers"], heads=c["heads"], kv_heads=max(1, c["heads"] // 8), dim=c["dim"], window=0, side_dim=0, vocab=c["vocab"],
+                ff_turns=[c["ff"] * 3 // 2, c["top"] * c["expert_ff"] + c["shared_ff"]])

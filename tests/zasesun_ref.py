@@ -107,7 +107,14 @@ def feed_forward(h, p, m):
     return expert_mlp(h, p, m) if m["kind"] == "moe" else gated_mlp(h, p)
 
 
-def forward(model, tokens):
+def margin(z, top):
+    """Distance of the last chosen logit from the first that is not."""
+    s = -np.sort(-z, axis=-1)
+    return s[:, top - 1] - s[:, top] if top < z.shape[-1] else np.full(z.shape[0], np.inf)
+
+
+def forward(model, tokens, margins=None):
+    """`margins` (a list) receives one array per expert layer: every token's margin()."""
     cfg = model["config"]
     W = {k: np.asarray(v, np.float64) for k, v in model["tensors"].items()}
     eps, mult, cap = cfg["norm"]["eps"], cfg["residual_mult"], cfg["logit_softcap"]
@@ -121,7 +128,10 @@ def forward(model, tokens):
         n = part(f"l{i}.")
         x = x + mult * rms_norm(latent_attention(rms_norm(x, n["norm1"], eps), part(f"l{i}.mix."), layer["mixer"], eps), n["norm1b"], eps)
         if layer["mlp"] is not None:
-            x = x + mult * rms_norm(feed_forward(rms_norm(x, n["norm2"], eps), part(f"l{i}.mlp."), layer["mlp"]), n["norm2b"], eps)
+            h, p = rms_norm(x, n["norm2"], eps), part(f"l{i}.mlp.")
+            if margins is not None and layer["mlp"]["kind"] == "moe":
+                margins.append(margin(h @ p["router"].T, layer["mlp"]["router"]["top"]))
+            x = x + mult * rms_norm(feed_forward(h, p, layer["mlp"]), n["norm2b"], eps)
         streams.append(x)
     logits = rms_norm(x, W["final.norm"], eps) @ W["embed"].T
     return cap * np.tanh(logits / cap), np.stack(streams)
