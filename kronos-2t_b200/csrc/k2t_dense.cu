@@ -105,9 +105,10 @@ cudaError_t gemv_nt(cudaStream_t s, const DenseView &m, const Act &x, uint32_t t
 // ------------------------------------------------------------------------------------------------ bf16 GEMM (tensor cores)
 // CTA = 128 rows x NT tokens.  Warp 4 streams operand tiles (one bulk copy of 16 KiB of weights and one of NT x 128 bytes of
 // activations per 64 columns; both lie in the operand layout already, so nothing touches them on the way), warp 5 issues four
-// tcgen05.mma (K 16 each) per stage and commits the stage back, warps 0 .. 3 read the accumulators out of tensor memory
-// (lane = row) and store fp32 rows: 32 consecutive outputs of a token per warp store.
-constexpr uint32_t GM_THREADS = 192;
+// tcgen05.mma (K 16 each) per stage and commits the stage back, warps 0 .. 3 and 6 .. 9 read the accumulators out of tensor memory
+// (lane = row, a quarter of the rows per warp, every second stretch of 32 tokens) and store: 32 consecutive outputs of a token per
+// warp store.
+constexpr uint32_t GM_THREADS = 320;
 constexpr uint32_t GM_A = DENSE_ROW_TILE * PANEL * 2;
 constexpr uint32_t GM_HEADER = 1024;
 constexpr uint32_t GM_WAIT_LIMIT = 1u << 22;
@@ -157,35 +158,46 @@ __device__ __forceinline__ void gm_ld32(uint32_t taddr, uint32_t (&v)[32]) {
         : "r"(taddr) : "memory");
 }
 
-// 32 sums per lane (lane = row, registers = tokens tok .. tok + n - 1) -> output.  Activations: neighbouring lanes swap halves, so
-// that a lane stores two columns (or one product of a pair) of every second token.
-__device__ __forceinline__ void gm_store(const DenseOut &o, uint32_t rows, uint32_t row, uint32_t tok, uint32_t n, uint32_t (&v)[32]) {
+// 32 sums per lane (lane = row, registers = tokens tok .. tok + n - 1, tok a multiple of eight) -> output.  Activations: neighbouring
+// lanes swap halves, so that a lane stores two columns (or one product of a pair) of every second token.  FULL: no token and no
+// row of the warp is beyond the end - stores without predicates, which take a fraction of the instructions.
+template <bool FULL> __device__ __forceinline__ void gm_store_part(const DenseOut &o, uint32_t rows, uint32_t row, uint32_t tok, uint32_t n, uint32_t (&v)[32]) {
     if (o.kind == Epi::Rows || o.kind == Epi::Softcap) {
-        if (row >= rows) return;
+        if (!FULL && row >= rows) return;
         float *p = o.rows + (size_t)tok * o.stride + row;
+        const uint32_t stride = (uint32_t)o.stride;
+        if (o.kind == Epi::Rows) {
 #pragma unroll
-        for (uint32_t t = 0; t < 32; ++t) {
-            float x = __uint_as_float(v[t]);
-            if (o.kind == Epi::Softcap) x = softcap(x, o.cap);
-            if (t < n) p[t * o.stride] = x;
+            for (uint32_t t = 0; t < 32; ++t)
+                if (FULL || t < n) p[t * stride] = __uint_as_float(v[t]);
+        } else {
+#pragma unroll
+            for (uint32_t t = 0; t < 32; ++t)
+                if (FULL || t < n) p[t * stride] = softcap(__uint_as_float(v[t]), o.cap);
         }
         return;
     }
-    const bool odd = (threadIdx.x & 1u) != 0;
+    const uint32_t odd = threadIdx.x & 1u, r = row & ~1u, k = o.kind == Epi::GeluGated ? r >> 1 : r, chunk = ((k >> 3) & 7u) ^ odd;
+    // element of (token tok + odd + t, column k) for even t: its chunk is chunk ^ (t & 7)
+    __nv_bfloat16 *p = static_cast<__nv_bfloat16 *>(o.act.p) + ((size_t)(k >> 6) * o.act.ld + tok + odd) * PANEL + (k & 7u);
 #pragma unroll
     for (uint32_t t = 0; t < 32; t += 2) {
         const float mine = __uint_as_float(odd ? v[t + 1] : v[t]), other = __shfl_xor_sync(0xffffffffu, __uint_as_float(odd ? v[t] : v[t + 1]), 1);
-        const uint32_t tt = t + (odd ? 1u : 0u), r = row & ~1u;
-        const float lo = odd ? other : mine, hi = odd ? mine : other;       // rows r and r + 1 of token tt
-        if (tt >= n || r >= rows) continue;
+        const float lo = odd ? other : mine, hi = odd ? mine : other;       // rows r and r + 1 of the token
+        if (!FULL && (t + odd >= n || r >= rows)) continue;
+        __nv_bfloat16 *q = p + t * PANEL + ((chunk ^ (t & 7u)) << 3);
         if (o.kind == Epi::GeluGated) {
-            act_store<false>(o.act, tok + tt, r >> 1, gelu_tanh(lo) * hi);
+            *q = __float2bfloat16_rn(gelu_tanh_fast(lo) * hi);
         } else {
             const float x = o.kind == Epi::Relu2 ? relu_squared(lo) : lo, y = o.kind == Epi::Relu2 ? relu_squared(hi) : hi;
-            if (r + 1 < rows) *reinterpret_cast<uint32_t *>(static_cast<__nv_bfloat16 *>(o.act.p) + panel_index(o.act.ld, tok + tt, r)) = pack_bf16(x, y);
-            else act_store<false>(o.act, tok + tt, r, x);
+            if (FULL || r + 1 < rows) *reinterpret_cast<uint32_t *>(q) = pack_bf16(x, y);
+            else *q = __float2bfloat16_rn(x);
         }
     }
+}
+__device__ __forceinline__ void gm_store(const DenseOut &o, uint32_t rows, uint32_t row, uint32_t tok, uint32_t n, uint32_t (&v)[32]) {
+    if (n == 32 && (row | 31u) < rows) gm_store_part<true>(o, rows, row, tok, n, v);
+    else gm_store_part<false>(o, rows, row, tok, n, v);
 }
 
 template <int NT, bool GROUPED>
@@ -279,12 +291,12 @@ __global__ void __launch_bounds__(GM_THREADS) dense_gemm_kernel(const GemmArgs a
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         ok = ok && *s_abort == 0;
         if (!ok && lane == 0 && a.err_flag != nullptr) atomicExch(a.err_flag, 1u);
-        const uint32_t row = row0 + warp * 32 + lane;
+        const uint32_t quarter = warp & 3u, row = row0 + quarter * 32 + lane;          // a warp reaches the tensor-memory lanes of its number mod 4
 #pragma unroll 1
-        for (uint32_t c = 0; c < NT; c += 32) {
+        for (uint32_t c = warp < 4 ? 0 : 32; c < NT; c += 64) {
             if (tok0 + c >= tok_end || !ok) break;
             uint32_t v[32];
-            gm_ld32(tmem + ((warp * 32u) << 16) + c, v);
+            gm_ld32(tmem + ((quarter * 32u) << 16) + c, v);
             gm_store(a.out, a.rows, row, tok0 + c, min(32u, tok_end - tok0 - c), v);
         }
     }
@@ -412,13 +424,15 @@ cudaError_t launch_dense_out(cudaStream_t s, const DeviceMatrix &dm, const Act &
     if (dm.geom.fmt != FMT_DENSE16) return cudaErrorInvalidValue;
     if (n_tok >= DENSE_TC_MIN) {
         const GemmArgs a{static_cast<const uint8_t *>(m.base), static_cast<const uint8_t *>(x.p), m.rows, m.rows_pad, m.panels, x.ld, n_tok, out, err_flag, nullptr, nullptr, nullptr};
-        // widest token tile that does not leave SMs idle: relative time of a tile against the waves of the grid
-        static const struct { uint32_t nt; float cost; } tiles[4] = {{256, 1.0f}, {128, 0.55f}, {64, 0.34f}, {32, 0.25f}};
+        // token tile by the time of the grid's waves (measured, in units of a 256-token wave): tiles up to 128 tokens run two CTAs
+        // per SM, so that one's stores overlap the other's products; activations cost the store phase more than fp32 rows
+        static const struct { uint32_t nt; float alone, wave; } tiles[4] = {{256, 1.0f, 1.0f}, {128, 0.88f, 1.12f}, {64, 0.86f, 0.78f}, {32, 0.85f, 0.70f}};
         uint32_t best = 32;
         float best_t = 1e30f;
         for (const auto &c : tiles) {
-            const uint32_t ctas = (m.rows_pad / DENSE_ROW_TILE) * ((n_tok + c.nt - 1) / c.nt);
-            const float t = (float)((ctas + sm_count - 1) / sm_count) * c.cost;
+            const uint32_t ctas = (m.rows_pad / DENSE_ROW_TILE) * ((n_tok + c.nt - 1) / c.nt), slots = (uint32_t)sm_count * (c.nt == 256 ? 1u : 2u);
+            float t = ctas <= (uint32_t)sm_count ? c.alone : (float)((ctas + slots - 1) / slots) * c.wave;
+            if (c.nt == 256 && out.kind != Epi::Rows) t *= 1.15f;
             if (t < best_t) { best_t = t; best = c.nt; }
         }
         *launches = 1;

@@ -66,6 +66,10 @@ template <bool F32, bool SHARED = false> __device__ __forceinline__ float row_do
 __device__ __forceinline__ float gelu_tanh(float z) {
     return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
+// the same to bf16 accuracy and better, for values that are rounded to bf16 next
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+    return __fdividef(z, 1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
 __device__ __forceinline__ float relu_squared(float z) { const float r = fmaxf(z, 0.0f); return r * r; }
 __device__ __forceinline__ float softcap(float z, float cap) { return cap * tanhf(z / cap); }
 // sum of row r (and, for pairs, of row r + 1 behind an even r) of token t -> output

@@ -476,26 +476,39 @@ __global__ void __launch_bounds__(VL_THREADS) latent_value_kernel(const SplitPar
 }
 
 // ------------------------------------------------------------------------------------------------ prompts, bf16
-// queries as operand panels: per head the unrotated part, then the rotated one, each padded to whole panels with zeros
+// queries as operand panels: per head the unrotated part, then the rotated one, each padded to whole panels with zeros; thread = one
+// 16-byte chunk.  ALIGNED: rows and parts start at multiples of four floats.
+template <bool ALIGNED>
 __global__ void __launch_bounds__(256) latent_query_kernel(const LatentAttnArgs a, uint32_t n_tok) {
     const LatentShape &d = a.d;
-    const uint32_t dc = latent_head_cols(d.dim), rc = latent_head_cols(d.rot_dim), per = dc + rc, t = blockIdx.y, pairs = d.heads * per / 2;
+    const uint32_t dc = latent_head_cols(d.dim), per = dc + latent_head_cols(d.rot_dim), t = blockIdx.y, chunks = d.heads * per / 8;
     pdl_wait();
     pdl_trigger();
     const float *cs = a.rot + (size_t)(__ldcg(a.pos) + t) * d.rot_dim;
-    for (uint32_t i = blockIdx.x * 256 + threadIdx.x; i < pairs; i += gridDim.x * 256) {
-        const uint32_t h = i / (per / 2), k = i % (per / 2) * 2;
-        const float *q = a.q + t * a.q_stride + h * (d.dim + d.rot_dim);
-        float x = 0.0f, y = 0.0f;
-        if (k < dc) {
-            if (k < d.dim) x = __ldcg(q + k);
-            if (k + 1 < d.dim) y = __ldcg(q + k + 1);
-        } else if (k - dc < d.rot_dim) {
-            const float u = __ldcg(q + d.dim + k - dc), v = __ldcg(q + d.dim + k - dc + 1), c = __ldg(cs + k - dc), s = __ldg(cs + k - dc + 1);
-            x = u * c - v * s;
-            y = v * c + u * s;
+    for (uint32_t i = blockIdx.x * 256 + threadIdx.x; i < chunks; i += gridDim.x * 256) {
+        const uint32_t h = i / (per / 8), k = i % (per / 8) * 8;
+        const bool rot = k >= dc;
+        const uint32_t k0 = rot ? k - dc : k, n = rot ? d.rot_dim : d.dim;          // elements k0 .. k0 + 7 of a part of n
+        const float *q = a.q + t * a.q_stride + h * (d.dim + d.rot_dim) + (rot ? d.dim : 0) + k0;
+        float v[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
+        if (ALIGNED && k0 + 8 <= n) {
+            const float4 x = __ldcg(reinterpret_cast<const float4 *>(q)), y = __ldcg(reinterpret_cast<const float4 *>(q) + 1);
+            v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+        } else {
+#pragma unroll
+            for (uint32_t j = 0; j < 8; ++j)
+                if (k0 + j < n) v[j] = __ldcg(q + j);
         }
-        *reinterpret_cast<uint32_t *>(static_cast<__nv_bfloat16 *>(a.q_rows.p) + panel_index(a.q_rows.ld, t, h * per + k)) = pack_bf16(x, y);
+        if (rot)
+#pragma unroll
+            for (uint32_t j = 0; j < 8; j += 2)
+                if (k0 + j < n) {
+                    const float c = __ldg(cs + k0 + j), s = __ldg(cs + k0 + j + 1), x = v[j], y = v[j + 1];
+                    v[j] = x * c - y * s;
+                    v[j + 1] = y * c + x * s;
+                }
+        *reinterpret_cast<uint4 *>(static_cast<__nv_bfloat16 *>(a.q_rows.p) + panel_index(a.q_rows.ld, t, h * per + k)) =
+            make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
     }
 }
 
@@ -738,7 +751,8 @@ __global__ void __launch_bounds__(FL_THREADS, 1) latent_flash_kernel(const Flash
             tc_fence_before();
             mbar_arrive(b_p + 8 * b);
         }
-        if (ok) ok = __all_sync(0xffffffffu, fl_wait(b_o, (n_tiles - 1) & 1u, s_abort));
+        // the last update by a barrier of its own: the phases of b_o may still be two behind here, and a parity tells only neighbours apart
+        if (ok) ok = __all_sync(0xffffffffu, fl_wait(b_end, 0u, s_abort) && *s_abort == 0);
         tc_fence_after();
         if (ok) {
             const float inv = 1.0f / l;
@@ -861,8 +875,9 @@ cudaError_t launch_latent_prompt(cudaStream_t s, const LatentAttnArgs &a, uint32
     const LatentShape &d = a.d;
     const FlashShape f = flash_shape(d);
     if (!latent_flash_fits(d) || n_tok > 65535u) return cudaErrorInvalidValue;
-    const uint32_t pairs = d.heads * (latent_head_cols(d.dim) + latent_head_cols(d.rot_dim)) / 2;
-    cudaError_t e = launch_kernel(latent_query_kernel, dim3(std::min(8u, (pairs + 255) / 256), n_tok), dim3(256), 0, s, pdl, a, n_tok);
+    const uint32_t chunks = d.heads * (latent_head_cols(d.dim) + latent_head_cols(d.rot_dim)) / 8;
+    const bool aligned = d.dim % 4 == 0 && d.rot_dim % 4 == 0 && a.q_stride % 4 == 0;
+    cudaError_t e = launch_kernel(aligned ? latent_query_kernel<true> : latent_query_kernel<false>, dim3(std::min(8u, (chunks + 255) / 256), n_tok), dim3(256), 0, s, pdl, a, n_tok);
     if (e != cudaSuccess) return e;
     const FlashParams p{a, n_tok, f.pd, f.pr, f.pv, f.vn, f.tmem};
     return f.kt == 128 ? flash_launch<128>(s, p, f.smem, pdl) : flash_launch<64>(s, p, f.smem, pdl);

@@ -286,6 +286,22 @@ def test_sequences_follow_one_another(engine):
     assert np.array_equal(eng.forward_token_ids(b, want_all=True), alone)
 
 
+def test_repeats_bit_for_bit(engine):
+    """The kernels' order of additions is fixed: thirty repeats of a prompt in two portions, and of a few decoded tokens."""
+    model = mixed("wide")
+    eng = engine(model, "bfloat16")
+    toks = tokens_of(model, 260)
+
+    def run():
+        a = eng.forward_token_ids(toks[:150], want_all=True)
+        b = eng.forward_token_ids(toks[150:250], pos_start=150, want_all=True)
+        return np.concatenate([a, b, decoded(eng, toks, 250)])
+
+    first = run()
+    for _ in range(30):
+        assert np.array_equal(run(), first)
+
+
 def test_first_tokens(engine):
     model = mixed("uneven")
     for n in (1, 2, 3, 17, 64, 65):
