@@ -15,7 +15,8 @@ namespace {
 // panels are requested before the dependency wait, so a launch whose warps hold few panels has its whole matrix in flight
 // while the predecessor still runs
 // (four with four CTAs per SM, six with two: more bytes in flight where the rows give only few CTAs).
-template <int NT, int GV_PF>
+// ROWS: the output is fp32 rows.
+template <int NT, int GV_PF, bool ROWS>
 __global__ void __launch_bounds__(256, NT == 1 && GV_PF == 4 ? 4 : 2) dense_gemv_kernel(const uint4 *__restrict__ w, uint32_t rows, uint32_t rows_pad, uint32_t np, const uint4 *__restrict__ x,
                                                         uint32_t ld, uint32_t t0, uint32_t n_tok, const DenseOut out, uint32_t wk_log2) {
     __shared__ float s_part[8][8][NT];
@@ -77,6 +78,10 @@ __global__ void __launch_bounds__(256, NT == 1 && GV_PF == 4 ? 4 : 2) dense_gemv
         if (row >= rows || t0 + t >= n_tok) continue;
         float s = 0.0f, s1 = 0.0f;
         for (uint32_t k = 0; k < wk; ++k) s = __fadd_rn(s, s_part[g * wk + k][row_l][t]);
+        if (ROWS) {
+            out.rows[(size_t)(t0 + t) * out.stride + row] = s;
+            continue;
+        }
         if (out.kind == Epi::GeluGated && (row_l & 1u) == 0)
             for (uint32_t k = 0; k < wk; ++k) s1 = __fadd_rn(s1, s_part[g * wk + k][row_l + 1][t]);
         dense_store<false>(out, t0 + t, row, s, s1);
@@ -97,7 +102,9 @@ cudaError_t gemv_nt(cudaStream_t s, const DenseView &m, const Act &x, uint32_t t
         if (t < best) { best = t; wl = l; }
     }
     const uint32_t per = 8u >> wl, ctas = (groups + per - 1) / per;
-    auto k = NT == 1 && ctas <= 2u * (uint32_t)sm_count ? dense_gemv_kernel<NT, NT == 1 ? 6 : 4> : dense_gemv_kernel<NT, 4>;
+    const bool deep = NT == 1 && ctas <= 2u * (uint32_t)sm_count;
+    constexpr int DEEP = NT == 1 ? 6 : 4;
+    auto k = out.kind == Epi::Rows ? (deep ? dense_gemv_kernel<NT, DEEP, true> : dense_gemv_kernel<NT, 4, true>) : deep ? dense_gemv_kernel<NT, DEEP, false> : dense_gemv_kernel<NT, 4, false>;
     return launch_kernel(k, dim3(ctas), dim3(256), 0, s, pdl, static_cast<const uint4 *>(m.base), m.rows, m.rows_pad, m.panels,
                          static_cast<const uint4 *>(x.p), x.ld, t0, n_tok, out, wl);
 }
