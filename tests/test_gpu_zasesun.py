@@ -191,6 +191,23 @@ def test_a_key_seen_from_a_prompt_batch_behind_it(engine, dtype):
         assert e[50] < TOL[dtype] and e.max() < 2 * TOL[dtype]          # most weight of a noise token is its attention's, normed and doubled
 
 
+@pytest.mark.parametrize("heads", [4, 70])
+def test_long_context_by_both_ways(engine, heads):
+    """Nine thousand positions: splits of several tiles, prompt batches that follow one another.  A prompt's last tokens (keys and
+    values expanded) against the same tokens decoded (in latent space); the key far back is what the last one looks at."""
+    model = zm.pointer(heads=heads)
+    eng = engine(model, "bfloat16", max_seq=9100)
+    toks = np.random.default_rng(1).integers(3, 40, 9000)
+    toks[[5, -1]] = 1, 2
+    eng.forward_token_ids(toks[:8900])
+    tail = eng.forward_token_ids(toks[8900:], pos_start=8900, want_all=True)
+    eng.forward_token_ids(toks[:8996])
+    assert fm.error(decoded(eng, toks, 8996), tail[96:]).max() < 3e-2
+    toks[5] = 9
+    eng.forward_token_ids(toks[:8999])
+    assert fm.error(decoded(eng, toks, 8999), tail[99:]).max() > 0.2
+
+
 def planted(model, change):
     """Error that a restatement with `change` applied to its configuration or tensors would show."""
     other = copy.deepcopy(model)
