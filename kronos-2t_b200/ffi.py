@@ -356,7 +356,7 @@ class Engine:
     qkv, o, gate_up, down}], final_norm, lm_head, rope [max_seq][head_dim], embed_bf16 (or None = tied).
 
     A spec with `blocks` describes an unquantized model block by block (kronos_cuda_engine_create_blocks): cfg {hidden, vocab,
-    max_seq, eps, side_dim, precision 16 | 32}, blocks [{mixer, heads, dim, .. as the fields of KronosCudaBlockDesc; vectors fp32,
+    max_seq, eps, side_dim, residual_mult, logit_softcap, precision 16 | 32}, blocks [{mixer, heads, dim, .. as the fields of KronosCudaBlockDesc; vectors fp32,
     matrices bf16 bit patterns (precision 16) or fp32}], final_norm, head, embed and side_embed (bf16 bit patterns)."""
 
     def __init__(self, ctx, spec):
